@@ -13,6 +13,7 @@ from .dodonex import DodonexConfig
 from .numuzen import NumuzenConfig
 from .fusolix import FusolixConfig
 from .kilatar import KilatarConfig
+from .tekarax import TekaraxConfig
 
 __all__ = [
     "DodonexConfig",
@@ -26,6 +27,7 @@ __all__ = [
     "PartSpec",
     "Qwen2Config",
     "ScheduleEntry",
+    "TekaraxConfig",
     "architecture_name",
     "ceil_div",
     "config_class_for",

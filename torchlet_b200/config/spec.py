@@ -77,12 +77,14 @@ class ScheduleEntry:
     names an earlier entry, whose cache it then reads without writing.  ``add_embedding``: before this
     execution the embedding output (the stream as it entered the first layer) is added to the stream
     (a model that runs a stretch of its layers several times feeds its input in again before each
-    further pass).
+    further pass).  ``add_row`` = r: row r of the table ``ModelSpec.stream_rows_name`` is added to every token's stream
+    before this execution (a vector that tells the passes of a looped stretch apart).
     """
 
     layer: int
     cache_from: Optional[int] = None
     add_embedding: bool = False
+    add_row: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -106,6 +108,9 @@ class ModelSpec:
     # a norm of the embedding rows (after the scale) before the first layer; its tensors lie below the prefix
     embedding_norm: Optional[PartSpec] = None
     embedding_norm_prefix: str = "embedding_norm."
+    # a tensor [stream_rows, hidden] whose rows schedule entries add to the stream (``ScheduleEntry.add_row``)
+    stream_rows_name: Optional[str] = None
+    stream_rows: int = 0
 
     def validate(self) -> None:
         if not self.layers:
@@ -114,7 +119,11 @@ class ModelSpec:
             raise ValueError("the layer schedule is empty")
         if self.streams is not None and any(entry.add_embedding for entry in self.schedule):
             raise ValueError("adding the embedding output again is not built for several residual streams")
+        if self.streams is not None and any(entry.add_row is not None for entry in self.schedule):
+            raise ValueError("adding a row to the stream is not built for several residual streams")
         for i, entry in enumerate(self.schedule):
+            if entry.add_row is not None and (self.stream_rows_name is None or not 0 <= entry.add_row < self.stream_rows):
+                raise ValueError(f"schedule entry {i} adds row {entry.add_row} of a table of {self.stream_rows} rows")
             if not 0 <= entry.layer < len(self.layers):
                 raise ValueError(
                     f"schedule entry {i} names layer {entry.layer}, "

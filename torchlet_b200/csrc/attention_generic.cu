@@ -7,7 +7,7 @@
 // sum are float32; T is the storage type of queries, pages and output.
 //
 // Options: ``softcap`` > 0 bounds a score, s <- softcap tanh(s / softcap); ``sink`` adds one to the
-// softmax's denominator (a key of score 0 that has no value); ``gate`` (float32 rows) multiplies the
+// softmax's denominator (a key of score 0 that has no value), or with ``sink_values`` exp(sink_values[head]); ``gate`` (float32 rows) multiplies the
 // output element by element with sigmoid(gate).
 //
 // This is the true 32-bit kernel and the any-size bfloat16 kernel (head_dim up to 256: keys are
@@ -36,7 +36,7 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
                          const int* __restrict__ token_req, const int* __restrict__ positions,
                          T* __restrict__ out, int out_stride, int tokens, int nh, int nkv, int d,
                          int page_size, int window, float scale, int num_pages, float softcap, int sink,
-                         const float* __restrict__ gate, int gate_stride, int wide) {
+                         const float* __restrict__ sink_values, const float* __restrict__ gate, int gate_stride, int wide) {
   tl::pdl_wait();               // everything before us in the stream is complete and visible
   tl::pdl_launch_dependents();  // the next kernel may start its own prologue
 
@@ -58,9 +58,9 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
   const size_t k_off = (size_t)kvh * page_size * d;
   const size_t v_off = ((size_t)nkv + kvh) * page_size * d;
 
-  // the sink is a key of score 0 and no value that every query sees: the running maximum starts
-  // at 0 with a weight of exp(0) in the denominator
-  float m = sink ? 0.f : -INFINITY, l = sink ? 1.f : 0.f;
+  // the sink is a key of a given score (0, or the head's own number) and no value that every query sees: the running
+  // maximum starts at that score with a weight of exp(0) in the denominator
+  float m = sink ? (sink_values ? sink_values[h] : 0.f) : -INFINITY, l = sink ? 1.f : 0.f;
   float acc[MAX_D / 32];
 #pragma unroll
   for (int c = 0; c < MAX_D / 32; ++c) acc[c] = 0.f;
@@ -131,7 +131,8 @@ extern "C" int tl_attention_generic(const void* q, int q_stride, const void* pag
                                     const int* block_table, int table_width, const int* token_req,
                                     const int* positions, void* out, int out_stride, int tokens,
                                     int nh, int nkv, int d, int page_size, int window, float scale,
-                                    int num_pages, float softcap, int sink, const float* gate, int gate_stride,
+                                    int num_pages, float softcap, int sink, const float* sink_values,
+                                    const float* gate, int gate_stride,
                                     cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (d <= 0 || d > MAX_D || nkv <= 0 || nh % nkv || page_size <= 0) return TL_ERR_UNSUPPORTED;
@@ -142,11 +143,11 @@ extern "C" int tl_attention_generic(const void* q, int q_stride, const void* pag
     tl::launch_kernel(attention_generic_kernel<float>, blocks, WARPS * 32, 0, stream, 
         (const float*)q, q_stride, (const float*)pages, block_table, table_width, token_req,
         positions, (float*)out, out_stride, tokens, nh, nkv, d, page_size, window, scale, num_pages, softcap, sink,
-        gate, gate_stride, wide);
+        sink_values, gate, gate_stride, wide);
   else
     tl::launch_kernel(attention_generic_kernel<__nv_bfloat16>, blocks, WARPS * 32, 0, stream, 
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)pages, block_table, table_width,
         token_req, positions, (__nv_bfloat16*)out, out_stride, tokens, nh, nkv, d, page_size, window,
-        scale, num_pages, softcap, sink, gate, gate_stride, wide);
+        scale, num_pages, softcap, sink, sink_values, gate, gate_stride, wide);
   return TL_LAUNCH_CHECK();
 }

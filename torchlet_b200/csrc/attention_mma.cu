@@ -72,6 +72,7 @@ struct Params {
   // (float32 rows [tokens][>= nh D]: the output is multiplied by sigmoid(gate))
   float cap_inner, cap_outer;
   int sink;
+  const float* sink_values;  // the sink's score of every query head (null: 0); it is not scaled
   const float* gate;
   long long gate_stride;
   // a PRIOR softmax state of every (token, head), computed elsewhere over keys this kernel does not walk (summary
@@ -82,10 +83,14 @@ struct Params {
 };
 
 __device__ __forceinline__ float capped_tanh(float x) { return 1.f - 2.f / (__expf(2.f * x) + 1.f); }
-// The softmax denominator with the sink's share: a key of score 0 against the running maximum m (log2 units).
-template <bool EXTRAS> __device__ __forceinline__ float with_sink(const Params& p, float l, float m) {
+// A head's sink score in log2 units.
+__device__ __forceinline__ float sink_log2(const float* sink_values, int head) {
+  return sink_values ? sink_values[head] * 1.4426950408889634f : 0.f;
+}
+// The softmax denominator with the sink's share: a key of that score against the running maximum m (log2 units).
+template <bool EXTRAS> __device__ __forceinline__ float with_sink(const Params& p, int head, float l, float m) {
   if constexpr (!EXTRAS) return l;
-  return (p.sink && m != -INFINITY) ? l + exp2f(-m) : l;
+  return (p.sink && m != -INFINITY) ? l + exp2f(sink_log2(p.sink_values, head) - m) : l;
 }
 // The factors that bring a row's own state (max m) and its prior (max prior.x) to their common max, which replaces m.
 struct PriorFactors { float own, theirs, sum; };
@@ -585,7 +590,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p)
         acc = acc * pf.own + prior_value<EXTRAS>(p, pf, token, head, D, c);
         l = l * pf.own + pf.sum;
         p.out[(size_t)token * p.out_stride + (size_t)head * D + c] =
-            __float2bfloat16_rn(acc / with_sink<EXTRAS>(p, l, m_all) * gate_of<EXTRAS>(p, token, head, D, c));
+            __float2bfloat16_rn(acc / with_sink<EXTRAS>(p, head, l, m_all) * gate_of<EXTRAS>(p, token, head, D, c));
       }
     }
     if (p.splits > 1 && p.arrivals) {
@@ -646,7 +651,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p)
             acc.z = acc.z * pf.own + prior_value<EXTRAS>(p, pf, tok0, kvh * g + r, D, c + 2);
             acc.w = acc.w * pf.own + prior_value<EXTRAS>(p, pf, tok0, kvh * g + r, D, c + 3);
           }
-          const float inv = 1.f / with_sink<EXTRAS>(p, l, m_ref);
+          const float inv = 1.f / with_sink<EXTRAS>(p, kvh * g + r, l, m_ref);
           if (EXTRAS && p.gate) {
             const int head = kvh * g + r;
             acc.x *= gate_of<EXTRAS>(p, tok0, head, D, c);
@@ -669,7 +674,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p)
       const int token = tok0 + row / g, head = kvh * g + row % g;
       float m_row = m_run[h];
       const PriorFactors pf = prior_of<EXTRAS>(p, token, head, m_row);
-      const float inv = 1.f / with_sink<EXTRAS>(p, l_run[h] * pf.own + pf.sum, m_row);
+      const float inv = 1.f / with_sink<EXTRAS>(p, head, l_run[h] * pf.own + pf.sum, m_row);
       __nv_bfloat16* dst = p.out + (size_t)token * p.out_stride + (size_t)head * D + (lane & 3) * 2;
 #pragma unroll
       for (int i = 0; i < DTILES; ++i) {
@@ -695,7 +700,7 @@ attention_combine_kernel(const float* __restrict__ part_acc, const float* __rest
                          const int* __restrict__ tile_req, const int* __restrict__ req_indptr,
                          const int* __restrict__ kv_before, int window,
                          __nv_bfloat16* __restrict__ out, long long out_stride, int nh, int grid_splits, int sink,
-                         const float* __restrict__ gate, long long gate_stride, const float* __restrict__ prior_ml,
+                         const float* __restrict__ sink_values, const float* __restrict__ gate, long long gate_stride, const float* __restrict__ prior_ml,
                          const float* __restrict__ prior_acc) {
   tl::pdl_launch_dependents();  // the next kernel may start its prologue (it waits for us before it reads our output)
   tl::pdl_wait();               // everything before us in the stream is complete and visible
@@ -732,7 +737,7 @@ attention_combine_kernel(const float* __restrict__ part_acc, const float* __rest
         m_all = m_ref = top;
       }
     }
-    if (sink && m_all != -INFINITY) l += exp2f(-m_ref);  // the sink's share of the denominator
+    if (sink && m_all != -INFINITY) l += exp2f(sink_log2(sink_values, head) - m_ref);  // the sink's share of the denominator
     if (c == 0) {
       total[0] = l;
       total[1] = own;
@@ -891,8 +896,8 @@ int tl_attention_mma_error() {
 // portions' attention (tl_attention_tc), which neither reads nor writes anything this call writes;
 // this grid then starts beside it on the SMs it leaves idle and waits for it only at its end.
 // pages: one cache layer [num_pages][2][nkv][page_size][d].
-// softcap > 0: scores are capped, s <- softcap tanh(s / softcap); sink: one is added to the softmax's
-// denominator; gate (float32 [tokens][gate_stride], or null): the output is multiplied by sigmoid(gate).
+// softcap > 0: scores are capped, s <- softcap tanh(s / softcap); sink: exp(sink_values[head]) (null:
+// one) is added to the softmax's denominator; gate (float32 [tokens][gate_stride], or null): the output is multiplied by sigmoid(gate).
 // prior_ml [tokens][nh][2], prior_acc [tokens][nh][d] (float32, or null): a softmax state over other keys that joins
 // every row where it is normalized (max in log2 units of the scaled score, sum, weighted values; max -inf: none).
 int tl_attention_mma_ex(const void* q, long long q_stride, const void* pages, long long num_pages, const int* block_table,
@@ -900,7 +905,8 @@ int tl_attention_mma_ex(const void* q, long long q_stride, const void* pages, lo
                         const int* req_indptr, const int* kv_before, const int* tile_req, const int* tile_row,
                         int tiles, void* out, long long out_stride, int tokens, int nh, int nkv, int d, int page_size,
                         int window, float scale, int rows16, int splits, void* workspace, long long workspace_bytes,
-                        int* arrivals, int late_wait, float softcap, int sink, const float* gate, long long gate_stride,
+                        int* arrivals, int late_wait, float softcap, int sink,
+                        const float* sink_values, const float* gate, long long gate_stride,
                         const float* prior_ml, const float* prior_acc, cudaStream_t stream) {
   if (tiles <= 0 || tokens <= 0) return 0;
   if ((d != 64 && d != 128) || nkv <= 0 || nh % nkv || page_size <= 0 || q_stride % 8 || out_stride % 4)
@@ -938,6 +944,7 @@ int tl_attention_mma_ex(const void* q, long long q_stride, const void* pages, lo
   p.cap_inner = softcap > 0.f ? scale / softcap : 0.f;
   p.cap_outer = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.sink = sink;
+  p.sink_values = sink_values;
   p.gate = gate;
   p.gate_stride = gate_stride;
   p.prior_ml = prior_acc ? prior_ml : nullptr;
@@ -952,10 +959,10 @@ int tl_attention_mma_ex(const void* q, long long q_stride, const void* pages, lo
   const int items = tiles * nh;
   if (d == 128)
     tl::launch_kernel(attention_combine_kernel<128>, items, 128, 0, stream, p.part_acc, p.part_ml, tile_req, req_indptr,
-                      kv_before, window, p.out, out_stride, nh, splits, sink, gate, gate_stride, p.prior_ml, p.prior_acc);
+                      kv_before, window, p.out, out_stride, nh, splits, sink, sink_values, gate, gate_stride, p.prior_ml, p.prior_acc);
   else
     tl::launch_kernel(attention_combine_kernel<64>, items, 64, 0, stream, p.part_acc, p.part_ml, tile_req, req_indptr,
-                      kv_before, window, p.out, out_stride, nh, splits, sink, gate, gate_stride, p.prior_ml, p.prior_acc);
+                      kv_before, window, p.out, out_stride, nh, splits, sink, sink_values, gate, gate_stride, p.prior_ml, p.prior_acc);
   return TL_LAUNCH_CHECK();
 }
 
@@ -967,7 +974,7 @@ int tl_attention_mma(const void* q, long long q_stride, const void* pages, long 
                      int* arrivals, int late_wait, cudaStream_t stream) {
   return tl_attention_mma_ex(q, q_stride, pages, num_pages, block_table, table_width, req_indptr, kv_before, tile_req,
                              tile_row, tiles, out, out_stride, tokens, nh, nkv, d, page_size, window, scale, rows16, splits,
-                             workspace, workspace_bytes, arrivals, late_wait, 0.f, 0, nullptr, 0, nullptr, nullptr, stream);
+                             workspace, workspace_bytes, arrivals, late_wait, 0.f, 0, nullptr, nullptr, 0, nullptr, nullptr, stream);
 }
 
 }  // extern "C"

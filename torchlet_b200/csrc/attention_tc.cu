@@ -79,6 +79,7 @@ struct Params {
   // (float32 rows [tokens][>= nh D]: the output is multiplied by sigmoid(gate))
   float cap_inner, cap_outer;
   int sink;
+  const float* sink_values;  // the sink's score of every query head (null: 0); it is not scaled
   const float* gate;
   long long gate_stride;
   // a PRIOR softmax state of every (token, head) over keys this kernel does not walk: prior_ml [tokens][nh][2] =
@@ -86,6 +87,11 @@ struct Params {
   const float* prior_ml;
   const float* prior_acc;
 };
+
+// A head's sink score in log2 units.
+__device__ __forceinline__ float sink_log2(const float* sink_values, int head) {
+  return sink_values ? sink_values[head] * 1.4426950408889634f : 0.f;
+}
 
 // tanh by the special-function unit (tanh.approx: relative error 2^-11, which the cap's factor turns into a
 // score error of a few thousandths where scores are far from the cap, and the weights are rounded to bfloat16)
@@ -514,7 +520,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) 
           prior = p.prior_acc + item * D;
         }
       }
-      if (EXTRAS && p.sink && m_ref != -INFINITY) l_sum += exp2f(-m_ref);  // the sink's share: a key of score 0
+      if (EXTRAS && p.sink && m_ref != -INFINITY) l_sum += exp2f(sink_log2(p.sink_values, kvh * g + row % g) - m_ref);  // the sink's share
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
       __nv_bfloat16* dst = nullptr;
       const float* gate = nullptr;
@@ -567,7 +573,7 @@ __global__ void __launch_bounds__(128)
 attention_tc_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
                           const int* __restrict__ token_req, const int* __restrict__ req_indptr,
                           __nv_bfloat16* __restrict__ out, long long out_stride, int tokens, int nh, int splits, int sink,
-                          const float* __restrict__ gate, long long gate_stride, const float* __restrict__ prior_ml,
+                          const float* __restrict__ sink_values, const float* __restrict__ gate, long long gate_stride, const float* __restrict__ prior_ml,
                           const float* __restrict__ prior_acc) {
   tl::pdl_launch_dependents();
   tl::pdl_wait();
@@ -604,7 +610,7 @@ attention_tc_merge_kernel(const float* __restrict__ part_acc, const float* __res
       m_all = top;
     }
   }
-  if (sink && m_all != -INFINITY) total += exp2f(-m_all);  // the sink's share: a key of score 0
+  if (sink && m_all != -INFINITY) total += exp2f(sink_log2(sink_values, head) - m_all);  // the sink's share
   const float inv = total > 0.f ? 1.f / total : 0.f;
   __nv_bfloat16* dst = out + (size_t)token * out_stride + (size_t)head * D + lane * PER;
   const float* gate_row = gate ? gate + (size_t)token * gate_stride + (size_t)head * D + lane * PER : nullptr;
@@ -649,7 +655,7 @@ template <int D>
 int launch_merge(const Params& p, const int* token_req, int tokens, cudaStream_t stream) {
   tl::launch_kernel(attention_tc_merge_kernel<D>, (tokens * p.nh + 3) / 4, 128, 0, stream, (const float*)p.part_acc,
                     (const float*)p.part_ml, token_req, p.req_indptr, p.out, p.out_stride, tokens, p.nh, p.splits, p.sink,
-                    p.gate, p.gate_stride, p.prior_ml, p.prior_acc);
+                    p.sink_values, p.gate, p.gate_stride, p.prior_ml, p.prior_acc);
   return TL_LAUNCH_CHECK();
 }
 
@@ -702,7 +708,7 @@ int tl_attention_tc(const void* q, long long q_stride, const void* pages, long l
                     const int* tile_req, const int* tile_row, int tiles, void* out, long long out_stride, int nh,
                     int nkv, int d, int page_size, int window, float scale, int splits, const int* token_req,
                     int tokens, void* workspace, long long workspace_bytes, int defer_merge, float softcap, int sink,
-                    const float* gate, long long gate_stride, const float* prior_ml, const float* prior_acc,
+                    const float* sink_values, const float* gate, long long gate_stride, const float* prior_ml, const float* prior_acc,
                     cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (splits < 1 || splits > 64) return TL_ERR_UNSUPPORTED;
@@ -735,6 +741,7 @@ int tl_attention_tc(const void* q, long long q_stride, const void* pages, long l
   p.cap_inner = softcap > 0.f ? scale / softcap : 0.f;
   p.cap_outer = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.sink = sink;
+  p.sink_values = sink_values;
   p.gate = gate;
   p.gate_stride = gate_stride;
   p.prior_ml = prior_acc ? prior_ml : nullptr;
@@ -755,7 +762,7 @@ int tl_attention_tc(const void* q, long long q_stride, const void* pages, long l
 // token_req and workspace as that call.
 int tl_attention_tc_merge(const int* req_indptr, void* out, long long out_stride, int nh, int d, int splits,
                           const int* token_req, int tokens, void* workspace, long long workspace_bytes, int sink,
-                          const float* gate, long long gate_stride, const float* prior_ml, const float* prior_acc,
+                          const float* sink_values, const float* gate, long long gate_stride, const float* prior_ml, const float* prior_acc,
                           cudaStream_t stream) {
   if (splits <= 1 || tokens <= 0) return 0;
   if ((d != 64 && d != 128) || !token_req || !workspace || out_stride % 8 ||
@@ -769,6 +776,7 @@ int tl_attention_tc_merge(const int* req_indptr, void* out, long long out_stride
   p.nh = nh;
   p.splits = splits;
   p.sink = sink;
+  p.sink_values = sink_values;
   p.gate = gate;
   p.gate_stride = gate_stride;
   p.prior_ml = prior_acc ? prior_ml : nullptr;

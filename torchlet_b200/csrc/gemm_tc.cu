@@ -5,7 +5,7 @@
 // tiles of both operands into a ring of shared-memory stages with TMA; one thread issues
 // tcgen05.mma (UMMA with 128 or 256 rows, K = 16) from shared-memory descriptors into an
 // accumulator in tensor memory and commits each stage back to the producer; four warps
-// read the accumulator with tcgen05.ld and run the epilogue (bias -> bf16, accumulate into
+// read the accumulator with tcgen05.ld and run the epilogue (bias -> bf16, with the square of relu or without, accumulate into
 // the float32 residual stream, SwiGLU over 16-interleaved gate/up rows, or float32 logits).
 //
 //   gemm_tc_swapped_kernel     few tokens (decode, M <= 256): the 128 tile rows are WEIGHT
@@ -40,7 +40,15 @@ constexpr int UMMA_K = 16;
 constexpr int ROW_TILE_BYTES = BLOCK_P * BLOCK_K * 2;
 constexpr int THREADS = 192;
 
-enum Epilogue { EPI_STORE_BF16 = 0, EPI_ACCUM_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_F32 = 3 };
+enum Epilogue { EPI_STORE_BF16 = 0, EPI_ACCUM_F32 = 1, EPI_SWIGLU_BF16 = 2, EPI_STORE_F32 = 3, EPI_RELU2_BF16 = 4 };
+
+// bf16 output: what is rounded (the square of relu with EPI_RELU2_BF16).
+__host__ __device__ __forceinline__ bool stores_bf16(int epilogue) { return epilogue == EPI_STORE_BF16 || epilogue == EPI_RELU2_BF16; }
+__device__ __forceinline__ float activated(int epilogue, float v) {
+  if (epilogue != EPI_RELU2_BF16) return v;
+  const float r = fmaxf(v, 0.f);
+  return r * r;
+}
 
 __device__ int g_error_word = 0;
 
@@ -139,7 +147,9 @@ __device__ __forceinline__ void epilogue_chunk(const Params& p, int m, int n0, c
 #pragma unroll
     for (int j = 0; j < 8; ++j) r[j] = v[c + j] + ((p.bias && n + j < N) ? p.bias[n + j] : 0.f);
     const bool full = n + 8 <= N;
-    if (p.epilogue == EPI_STORE_BF16) {
+    if (stores_bf16(p.epilogue)) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) r[j] = activated(p.epilogue, r[j]);
       __nv_bfloat16* o = (__nv_bfloat16*)p.out + (size_t)m * p.ldo + n;
       if (full && ((reinterpret_cast<uintptr_t>(o) & 15) == 0)) {
         uint32_t packed[4];
@@ -388,8 +398,8 @@ gemm_tc_swapped_kernel(const __grid_constant__ CUtensorMap map_row, const __grid
           const int m = col0 + c + j;
           if (m >= p.cols) break;
           const float r = v[j] + b;
-          if (p.epilogue == EPI_STORE_BF16)
-            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldo + row] = __float2bfloat16_rn(r);
+          if (stores_bf16(p.epilogue))
+            ((__nv_bfloat16*)p.out)[(size_t)m * p.ldo + row] = __float2bfloat16_rn(activated(p.epilogue, r));
           else if (p.epilogue == EPI_ACCUM_F32)
             ((float*)p.out)[(size_t)m * p.ldo + row] += r;
           else
@@ -781,8 +791,8 @@ __global__ void splitk_finish_kernel(const float* __restrict__ partial, int spli
   float v = 0.f;
   for (int s = 0; s < splits; ++s) v += partial[s * plane + (size_t)m * N + c];
   if (bias) v += bias[c];
-  if (epilogue == EPI_STORE_BF16)
-    ((__nv_bfloat16*)out)[(size_t)m * ldo + c] = __float2bfloat16_rn(v);
+  if (stores_bf16(epilogue))
+    ((__nv_bfloat16*)out)[(size_t)m * ldo + c] = __float2bfloat16_rn(activated(epilogue, v));
   else if (epilogue == EPI_ACCUM_F32)
     ((float*)out)[(size_t)m * ldo + c] += v;
   else
@@ -1038,7 +1048,7 @@ int tl_gemm_tc_error() {
 // out (+)= x[M, K] . w[N, K]^T.  x and w bfloat16 with K contiguous, ldx/ldw elements
 // between rows (multiples of 8, bases 16-byte aligned).  epilogue: 0 bf16 out + bias,
 // 1 float32 out += result, 2 SwiGLU over 16-interleaved gate/up rows of w -> bf16
-// [M, N/2], 3 float32 out.  workspace: float32 scratch of at least tl_gemm_tc_plan bytes.
+// [M, N/2], 3 float32 out, 4 bf16 out of relu(result + bias)^2.  workspace: float32 scratch of at least tl_gemm_tc_plan bytes.
 static int gemm_tc_impl(const void* x, const void* w, const float* bias, void* out, long long ldo, int epilogue, int M,
                         int N, int K, long long ldx, long long ldw, void* workspace, long long workspace_bytes,
                         int defer, int* splits_out, float glu_limit, float glu_alpha, cudaStream_t stream,
@@ -1076,7 +1086,7 @@ static int gemm_tc_impl(const void* x, const void* w, const float* bias, void* o
                         int defer, int* splits_out, float glu_limit, float glu_alpha, cudaStream_t stream,
                         const float* row_scale) {
   if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || epilogue < 0 || epilogue > 3) return TL_ERR_UNSUPPORTED;
+  if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || epilogue < 0 || epilogue > 4) return TL_ERR_UNSUPPORTED;
   if (epilogue == EPI_SWIGLU_BF16 && N % 32) return TL_ERR_UNSUPPORTED;
   if (epilogue != EPI_SWIGLU_BF16 && row_scale) return TL_ERR_UNSUPPORTED;
   const Plan plan = make_plan(M, N, K);

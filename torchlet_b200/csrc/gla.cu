@@ -6,7 +6,12 @@
 // with a decay per key channel a = sigmoid(z)^(1/tau) = exp(logsigmoid(z) / tau), z = W2 l + b, where
 // l is a low-rank projection of the layer's input.  Everything here is float32, also in the bfloat16
 // engine: the projections arrive as float32 rows
-//   proj[t] = [ q (H D) | k (H D) | v (H V) | g (H V) | l (rank) ].
+//   proj[t] = [ q (H D) | k (H D) | v (H V) | g (H V) | l (rank) ],
+// or with q, k and v in planes of their own (the scan takes the distances from q to k and to v).
+//
+// A time-mixing recurrence with a bonus for the current token is the same scan with one more vector u per head:
+//   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t,      S_t = diag(a_t) S_(t-1) + k_t v_t^T,
+// whose decay is a = exp(-exp(z)), z = W2 tanh(l) + b.
 //
 // Three kernels:
 //   decay   one block per (8 tokens, 128 channels): a of every key channel;
@@ -17,7 +22,7 @@
 //           is read at the start and written back at the end, so a prompt cut into portions, or
 //           decoded token by token, runs the same additions in the same order as the whole prompt;
 //   finish  one warp per (token, head): o / rms(o) * weight * silu(g) in the compute type (the
-//           weight covers one head and is shared by all).
+//           weight covers one head and is shared by all, or has every head's own numbers).
 #include <math.h>
 
 #include "common.cuh"
@@ -33,7 +38,7 @@ constexpr int DECAY_NT = 128;
 __global__ void __launch_bounds__(DECAY_NT)
 gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset, const float* __restrict__ w2t,
                  const float* __restrict__ bias, float* __restrict__ out, int tokens, int channels, int rank,
-                 float inv_tau) {
+                 float inv_tau) {  // inv_tau > 0: sigmoid(z)^(inv_tau); 0: exp(-exp(z)) of a tanh of the low-rank input
   tl::pdl_launch_dependents();
   tl::pdl_wait();
   extern __shared__ float low[];  // DECAY_TOKENS x rank
@@ -41,7 +46,8 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
   const int count = tokens - t0 < DECAY_TOKENS ? tokens - t0 : DECAY_TOKENS;
   for (int e = threadIdx.x; e < DECAY_TOKENS * rank; e += DECAY_NT) {
     const int tt = e / rank, j = e - tt * rank;
-    low[e] = tt < count ? proj[(size_t)(t0 + tt) * proj_stride + low_offset + j] : 0.f;
+    const float l = tt < count ? proj[(size_t)(t0 + tt) * proj_stride + low_offset + j] : 0.f;
+    low[e] = inv_tau > 0.f ? l : tanhf(l);
   }
   __syncthreads();
   const int c = blockIdx.y * DECAY_NT + threadIdx.x;
@@ -60,6 +66,10 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
   for (int tt = 0; tt < DECAY_TOKENS; ++tt) {
     if (tt >= count) break;
     const float x = z[tt] + b;
+    if (inv_tau == 0.f) {
+      out[(size_t)(t0 + tt) * channels + c] = expf(-expf(x));
+      continue;
+    }
     // log(sigmoid(x)) = min(x, 0) - log1p(exp(-|x|))
     const float logsig = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
     out[(size_t)(t0 + tt) * channels + c] = expf(logsig * inv_tau);
@@ -96,15 +106,18 @@ constexpr int STAGES = 4;
 // constant per head (``heads`` numbers; a retention), DECAY_TOKEN one number per (token, head) for all of the head's
 // key channels (a selective state space).  ``qk_heads``: q and k have that many heads (a divisor of ``heads``), head h
 // reading q/k head h / (heads / qk_heads); the rows are [ q (qk_heads D) | k (qk_heads D) | v (heads V) | ... ].
-constexpr int DECAY_ROWS = 0, DECAY_HEAD = 1, DECAY_TOKEN = 2;
+// DECAY_BONUS: rows like DECAY_ROWS, and ``bonus`` [heads * dim] weighs the current token's k v^T in its own output.
+// k stands ``k_offset`` numbers behind q, v ``v_offset``.
+constexpr int DECAY_ROWS = 0, DECAY_HEAD = 1, DECAY_TOKEN = 2, DECAY_BONUS = 3;
 template <int DK, bool VEC, int MODE>
 __global__ void __launch_bounds__(lanes_a_column(DK) * COLS)
 gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ decay,
                 const int* __restrict__ req_indptr, const int* __restrict__ slots, float* __restrict__ state,
-                float* __restrict__ out, int heads, int qk_heads, int dim, int vdim, int max_slots, float qscale) {
+                float* __restrict__ out, int heads, int qk_heads, int dim, int vdim, int max_slots, float qscale,
+                const float* __restrict__ bonus, long long k_offset, long long v_offset) {
   tl::pdl_launch_dependents();
   tl::pdl_wait();
-  constexpr bool FIXED = MODE != DECAY_ROWS;  // no decay row is staged
+  constexpr bool FIXED = MODE == DECAY_HEAD || MODE == DECAY_TOKEN;  // no decay row is staged
   constexpr int KS = lanes_a_column(DK);
   constexpr int PER = DK / KS;
   // a staged token: q, k, (a: only where the decay is a row a token), v, the token's decay number.  Without the a
@@ -119,7 +132,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
   const int cols_here = vdim - col0 < COLS ? vdim - col0 : COLS;
   const int part = tid % KS, col = col0 + tid / KS;
   const bool on = col < vdim;
-  const int hd = qk_heads * dim, hv = heads * vdim;
+  const int hv = heads * vdim;
   const int hq = h / (heads / qk_heads);  // the q/k head this head reads
   const int first = req_indptr[req], last = req_indptr[req + 1];
   const int slot = slots[req];
@@ -144,7 +157,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
         float* to;
         if (rest < 2 * qd) {  // q, k
           const int what = rest / qd, q4 = rest - what * qd;
-          src = proj + (size_t)t * proj_stride + what * hd + hq * dim + 4 * q4;
+          src = proj + (size_t)t * proj_stride + what * k_offset + hq * dim + 4 * q4;
           to = dst + tt * row + what * DK + 4 * q4;
         } else if (!FIXED && rest < 3 * qd) {
           const int q4 = rest - 2 * qd;
@@ -155,7 +168,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
           continue;
         } else {
           const int q4 = rest - (FIXED ? 2 : 3) * qd;
-          src = proj + (size_t)t * proj_stride + 2 * hd + h * vdim + col0 + 4 * q4;
+          src = proj + (size_t)t * proj_stride + v_offset + h * vdim + col0 + 4 * q4;
           to = dst + tt * row + VOFF + 4 * q4;
         }
         copy16(to, src);
@@ -169,7 +182,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
         float* to;
         if (rest < 2 * dim) {
           const int what = rest / dim, i = rest - what * dim;
-          src = proj + (size_t)t * proj_stride + what * hd + hq * dim + i;
+          src = proj + (size_t)t * proj_stride + what * k_offset + hq * dim + i;
           to = dst + tt * row + what * DK + i;
         } else if (!FIXED && rest < 3 * dim) {
           const int i = rest - 2 * dim;
@@ -180,7 +193,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
           to = dst + tt * row + VOFF + COLS;
         } else {
           const int i = rest - (FIXED ? 2 : 3) * dim;
-          src = proj + (size_t)t * proj_stride + 2 * hd + h * vdim + col0 + i;
+          src = proj + (size_t)t * proj_stride + v_offset + h * vdim + col0 + i;
           to = dst + tt * row + VOFF + i;
         }
         copy4(to, src);
@@ -200,6 +213,15 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
   for (int n = 0; n < PER; ++n) {
     const int i = 4 * ((n >> 2) * KS + part) + (n & 3);
     S[n] = (on && i < dim) ? mine[(size_t)i * vdim + col] : 0.f;
+  }
+
+  float U[MODE == DECAY_BONUS ? PER : 1];  // the bonus of the same key channels
+  if (MODE == DECAY_BONUS) {
+#pragma unroll
+    for (int n = 0; n < PER; ++n) {
+      const int i = 4 * ((n >> 2) * KS + part) + (n & 3);
+      U[n] = i < dim ? bonus[(size_t)h * dim + i] : 0.f;
+    }
   }
 
   const float head_decay = MODE == DECAY_HEAD ? decay[h] : 0.f;
@@ -224,6 +246,18 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
       for (int n = 0; n < PER / 4; ++n) {
         const float4 a = FIXED ? make_float4(fixed, fixed, fixed, fixed) : a4[n * KS + part];
         const float4 k = k4[n * KS + part], q = q4[n * KS + part];
+        if constexpr (MODE == DECAY_BONUS) {  // the output reads the state before the token joins it
+          const float kx = k.x * v, ky = k.y * v, kz = k.z * v, kw = k.w * v;
+          o0 = fmaf(q.x, fmaf(U[4 * n], kx, S[4 * n]), o0);
+          o1 = fmaf(q.y, fmaf(U[4 * n + 1], ky, S[4 * n + 1]), o1);
+          o2 = fmaf(q.z, fmaf(U[4 * n + 2], kz, S[4 * n + 2]), o2);
+          o3 = fmaf(q.w, fmaf(U[4 * n + 3], kw, S[4 * n + 3]), o3);
+          S[4 * n] = fmaf(a.x, S[4 * n], kx);
+          S[4 * n + 1] = fmaf(a.y, S[4 * n + 1], ky);
+          S[4 * n + 2] = fmaf(a.z, S[4 * n + 2], kz);
+          S[4 * n + 3] = fmaf(a.w, S[4 * n + 3], kw);
+          continue;
+        }
         S[4 * n] = fmaf(k.x, v, a.x * S[4 * n]);
         S[4 * n + 1] = fmaf(k.y, v, a.y * S[4 * n + 1]);
         S[4 * n + 2] = fmaf(k.z, v, a.z * S[4 * n + 2]);
@@ -255,7 +289,7 @@ constexpr int FINISH_WARPS = 4;
 template <typename T>
 __global__ void __launch_bounds__(FINISH_WARPS * 32)
 gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj, int proj_stride, int gate_offset,
-                  const float* __restrict__ weight, T* __restrict__ out, long long items, int heads, int vdim,
+                  const float* __restrict__ weight, int weight_stride, T* __restrict__ out, long long items, int heads, int vdim,
                   float eps) {
   tl::pdl_launch_dependents();
   tl::pdl_wait();
@@ -273,7 +307,7 @@ gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj, i
   const float* gate = proj + (size_t)t * proj_stride + gate_offset + h * vdim;
   for (int i = lane; i < vdim; i += 32) {
     const float g = gate[i];
-    out[(size_t)t * hv + h * vdim + i] = from_float<T>(row[i] * inv * (weight ? weight[i] : 1.f) * (g / (1.f + expf(-g))));
+    out[(size_t)t * hv + h * vdim + i] = from_float<T>(row[i] * inv * (weight ? weight[h * weight_stride + i] : 1.f) * (g / (1.f + expf(-g))));
   }
 }
 
@@ -303,42 +337,46 @@ TL_DEBUG_READER(tl_gla_debug_error)
 extern "C" {
 
 // decay: float32 [tokens, channels] scratch; w2t: [rank, channels]; the low-rank input is
-// proj[t, low_offset : low_offset + rank].
+// proj[t, low_offset : low_offset + rank].  tau > 0: sigmoid(W2 l + bias)^(1 / tau); 0: exp(-exp(W2 tanh(l) + bias)).
 int tl_gla_decay(const float* proj, int proj_stride, int low_offset, const float* w2t, const float* bias, float* decay,
                  int tokens, int channels, int rank, float tau, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (channels <= 0 || rank <= 0 || rank > 1024 || !(tau > 0.f)) return TL_ERR_UNSUPPORTED;
+  if (channels <= 0 || rank <= 0 || rank > 1024 || !(tau >= 0.f)) return TL_ERR_UNSUPPORTED;
   dim3 grid((tokens + DECAY_TOKENS - 1) / DECAY_TOKENS, (channels + DECAY_NT - 1) / DECAY_NT);
   if (grid.y > 65535) return TL_ERR_UNSUPPORTED;
   tl::launch_kernel(gla_decay_kernel, grid, DECAY_NT, (size_t)DECAY_TOKENS * rank * sizeof(float), stream, proj,
-                    proj_stride, low_offset, w2t, bias, decay, tokens, channels, rank, 1.f / tau);
+                    proj_stride, low_offset, w2t, bias, decay, tokens, channels, rank, tau > 0.f ? 1.f / tau : 0.f);
   return TL_LAUNCH_CHECK();
 }
 
 // state: float32 [max_slots, heads, dim, vdim]; out: float32 [tokens, heads * vdim].
 // decay_mode: 0 ``decay`` holds [tokens, heads * dim] rows, 1 one constant per head, 2 [tokens, heads] (one number per
-// token and head).  qk_heads: how many heads q and k have (divides heads).
+// token and head), 3 rows and ``bonus`` [heads * dim].  k_offset, v_offset: how far k and v stand behind q.  qk_heads: how many heads q and k have (divides heads).
 int tl_gla_scan(const float* proj, int proj_stride, const float* decay, const int* req_indptr, const int* slots,
                 float* state, float* out, int requests, int heads, int qk_heads, int dim, int vdim, int max_slots,
-                float qscale, int decay_mode, cudaStream_t stream) {
+                float qscale, int decay_mode, const float* bonus, long long k_offset, long long v_offset,
+                cudaStream_t stream) {
   if (requests <= 0) return 0;
   if (dim <= 0 || dim > 256 || vdim <= 0 || vdim > 256 || heads > 65535) return TL_ERR_UNSUPPORTED;
-  if (qk_heads <= 0 || heads % qk_heads || decay_mode < 0 || decay_mode > 2) return TL_ERR_UNSUPPORTED;
-  const bool fixed_decay = decay_mode != DECAY_ROWS;
+  if (qk_heads <= 0 || heads % qk_heads || decay_mode < 0 || decay_mode > 3) return TL_ERR_UNSUPPORTED;
+  if ((decay_mode == DECAY_BONUS) != (bonus != nullptr)) return TL_ERR_UNSUPPORTED;
+  const bool fixed_decay = decay_mode == DECAY_HEAD || decay_mode == DECAY_TOKEN;
   dim3 grid(requests, heads, (vdim + COLS - 1) / COLS);
-  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && proj_stride % 4 == 0 && (qk_heads * dim) % 4 == 0 &&
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && proj_stride % 4 == 0 && k_offset % 4 == 0 && v_offset % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
                    (fixed_decay || (reinterpret_cast<uintptr_t>(decay) & 15) == 0);
 #define TL_SCAN_ONE(DK, VEC, MODE)                                                                                 \
   tl::launch_kernel(gla_scan_kernel<DK, VEC, MODE>, grid, lanes_a_column(DK) * COLS, 0, stream, proj, proj_stride, decay, req_indptr, \
-                    slots, state, out, heads, qk_heads, dim, vdim, max_slots, qscale)
+                    slots, state, out, heads, qk_heads, dim, vdim, max_slots, qscale, bonus, k_offset, v_offset)
 #define TL_SCAN(DK)                                                                \
   {                                                                                \
     if (vec && decay_mode == DECAY_HEAD) TL_SCAN_ONE(DK, true, DECAY_HEAD);        \
     else if (vec && decay_mode == DECAY_TOKEN) TL_SCAN_ONE(DK, true, DECAY_TOKEN); \
+    else if (vec && decay_mode == DECAY_BONUS) TL_SCAN_ONE(DK, true, DECAY_BONUS); \
     else if (vec) TL_SCAN_ONE(DK, true, DECAY_ROWS);                               \
     else if (decay_mode == DECAY_HEAD) TL_SCAN_ONE(DK, false, DECAY_HEAD);         \
     else if (decay_mode == DECAY_TOKEN) TL_SCAN_ONE(DK, false, DECAY_TOKEN);       \
+    else if (decay_mode == DECAY_BONUS) TL_SCAN_ONE(DK, false, DECAY_BONUS);       \
     else TL_SCAN_ONE(DK, false, DECAY_ROWS);                                       \
   }
   if (dim <= 16) TL_SCAN(16)
@@ -361,17 +399,17 @@ int tl_rotate_heads_f32(float* rows, int stride, const int* positions, const flo
   return TL_LAUNCH_CHECK();
 }
 
-int tl_gla_finish(const float* o, const float* proj, int proj_stride, int gate_offset, const float* weight, void* out,
+int tl_gla_finish(const float* o, const float* proj, int proj_stride, int gate_offset, const float* weight, int weight_stride, void* out,
                   int out_dtype, int tokens, int heads, int vdim, float eps, cudaStream_t stream) {
   const long long items = (long long)tokens * heads;
   if (items <= 0) return 0;
   const unsigned blocks = (unsigned)((items + FINISH_WARPS - 1) / FINISH_WARPS);
   if (out_dtype == TL_DTYPE_F32)
     tl::launch_kernel(gla_finish_kernel<float>, blocks, FINISH_WARPS * 32, 0, stream, o, proj, proj_stride,
-                      gate_offset, weight, (float*)out, items, heads, vdim, eps);
+                      gate_offset, weight, weight_stride, (float*)out, items, heads, vdim, eps);
   else
     tl::launch_kernel(gla_finish_kernel<__nv_bfloat16>, blocks, FINISH_WARPS * 32, 0, stream, o, proj, proj_stride,
-                      gate_offset, weight, (__nv_bfloat16*)out, items, heads, vdim, eps);
+                      gate_offset, weight, weight_stride, (__nv_bfloat16*)out, items, heads, vdim, eps);
   return TL_LAUNCH_CHECK();
 }
 

@@ -15,7 +15,8 @@
 //   attention   one warp per (token, head), keys in tiles of 32 consecutive ABSOLUTE positions,
 //               float32 scores, online softmax and sums: the order of every sum depends only on
 //               the token's position, never on the cut, the batch or the pages (the true 32-bit
-//               kernel and the any-size kernel);
+//               kernel and the any-size kernel); a sliding window or a chunked mask by the mask code of
+//               common.cuh;
 //   expand_o    one block per (8 tokens, head): out[t, h] = W_uv,h o_lat[t, h].
 // For many tokens the two per-head products run on the tensor cores instead (the mixer's choice).
 //
@@ -142,7 +143,7 @@ __global__ void __launch_bounds__(WARPS * 32)
 latent_attention_kernel(const T* __restrict__ q_abs, const T* __restrict__ pages, const int* __restrict__ block_table,
                         int table_width, const int* __restrict__ token_req, const int* __restrict__ positions,
                         T* __restrict__ out, int tokens, int heads, int dk, int dv, int page_size, float scale,
-                        int num_pages) {
+                        int num_pages, int window) {
   tl::pdl_wait();
   tl::pdl_launch_dependents();
   extern __shared__ float qs_all[];  // WARPS x dk
@@ -162,9 +163,10 @@ latent_attention_kernel(const T* __restrict__ q_abs, const T* __restrict__ pages
 #pragma unroll
   for (int c = 0; c < MAX_DV / 32; ++c) acc[c] = 0.f;
 
-  for (int start = 0; start <= pos; start += 32) {
+  const int lo = first_key(pos, window);
+  for (int start = lo & ~31; start <= pos; start += 32) {
     const int key = start + lane;
-    const bool valid = key <= pos;
+    const bool valid = key >= lo && key <= pos;
     float s = -INFINITY;
     size_t row_off = 0;
     if (valid) {
@@ -193,8 +195,9 @@ latent_attention_kernel(const T* __restrict__ q_abs, const T* __restrict__ pages
     m = new_m;
 #pragma unroll
     for (int c = 0; c < MAX_DV / 32; ++c) acc[c] *= corr;
+    const int first = lo > start ? lo - start : 0;
     const int last = pos - start < 31 ? pos - start : 31;
-    for (int j = 0; j <= last; ++j) {
+    for (int j = first; j <= last; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const size_t off = __shfl_sync(0xffffffffu, (unsigned long long)row_off, j);
       const T* vrow = pages + off;
@@ -326,7 +329,7 @@ int tl_latent_absorb_q(const float* q, int q_stride, const void* uk, int dtype, 
 
 int tl_latent_attention(const void* q_abs, const void* pages, int dtype, const int* block_table, int table_width,
                         const int* token_req, const int* positions, void* out, int tokens, int heads, int dk, int dv,
-                        int page_size, float scale, int num_pages, cudaStream_t stream) {
+                        int page_size, float scale, int num_pages, int window, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (dv <= 0 || dv > MAX_DV || dv > dk || dk > 2048) return TL_ERR_UNSUPPORTED;
   const long long items = (long long)tokens * heads;
@@ -336,7 +339,7 @@ int tl_latent_attention(const void* q_abs, const void* pages, int dtype, const i
 #define TL_LATENT(T, VEC)                                                                                       \
   tl::launch_kernel(latent_attention_kernel<T, VEC>, blocks, WARPS * 32, smem, stream, (const T*)q_abs,         \
                     (const T*)pages, block_table, table_width, token_req, positions, (T*)out, tokens, heads, dk, \
-                    dv, page_size, scale, num_pages)
+                    dv, page_size, scale, num_pages, window)
   if (dtype == TL_DTYPE_F32) {
     if (vec) TL_LATENT(float, true); else TL_LATENT(float, false);
   } else {

@@ -11,7 +11,8 @@
 // of the NCW warps of a row block meet in shared memory, P goes to shared memory in bfloat16, and
 // for O every warp reads all of P and the value columns [cw DVW, (cw + 1) DVW) that it accumulates
 // (DVW <= 128: 64 float registers a thread).  NCW = 1, 2, 4 for dv up to 128, 256, 512.
-// Rows of keys past the tile's last visible key are zero-filled (0 x stale NaN would be NaN).
+// Rows of keys outside what the tile's rows see (past the last row's own, before the first row's first under a window
+// or a chunked mask) are zero-filled (0 x stale NaN would be NaN).
 //
 // Requests that bring one token (decode) may split their keys over gridDim.y CTAs; every split
 // leaves an unnormalized partial result (O, max, sum) and a second kernel merges them.  How many
@@ -67,7 +68,7 @@ struct Args {
   __nv_bfloat16* out;
   float* part_o;         // [T heads][splits][dv]   (splits > 1)
   float* part_ml;        // [T heads][splits][2]
-  int table_width, heads, dk, dv, page_size, num_pages, tiles_per_req, splits;
+  int table_width, heads, dk, dv, page_size, num_pages, tiles_per_req, splits, window;
   float scale;
 };
 
@@ -97,11 +98,12 @@ latent_attention_mma_kernel(const Args a) {
   const int nrows = rows_total - row0 < ROWS ? rows_total - row0 : ROWS;
   const int kvb = a.kv_before[req];
   const int kv_end = kvb + (row0 + nrows - 1) / a.heads + 1;  // keys the tile's last row sees
+  const int kv_lo = first_key(kvb + row0 / a.heads, a.window);  // the first key the tile's first row sees
   const int key_tiles = (kv_end + KEYS - 1) / KEYS;
-  int tile_lo = 0, tile_hi = key_tiles;
+  int tile_lo = kv_lo / KEYS, tile_hi = key_tiles;
   if (a.splits > 1) {
-    const int per = (key_tiles + a.splits - 1) / a.splits;
-    tile_lo = split * per;
+    const int per = (key_tiles - tile_lo + a.splits - 1) / a.splits;
+    tile_lo += split * per;
     tile_hi = tile_lo + per < key_tiles ? tile_lo + per : key_tiles;
   }
   const int* table = a.block_table + (size_t)req * a.table_width;
@@ -126,6 +128,7 @@ latent_attention_mma_kernel(const Args a) {
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int r_lo = rw * 16 + g, r_hi = r_lo + 8;
   const int pos_lo = kvb + (row0 + r_lo) / a.heads, pos_hi = kvb + (row0 + r_hi) / a.heads;
+  const int from_lo = first_key(pos_lo, a.window), from_hi = first_key(pos_hi, a.window);
   const bool on_lo = r_lo < nrows, on_hi = r_hi < nrows;
   const bool warp_has_rows = rw * 16 < nrows;  // a tile of few rows (single tokens, few heads): the other warps only load
 
@@ -135,7 +138,7 @@ latent_attention_mma_kernel(const Args a) {
     for (int e = tid; e < KEYS * chunks; e += 128 * NCW) {
       const int r = e / chunks, c = e - r * chunks;
       const int key = key0 + r;
-      const bool valid = key < kv_end;
+      const bool valid = key >= kv_lo && key < kv_end;
       int page = 0;
       if (valid) {
         if (TL_DEBUG_OK(key / a.page_size < a.table_width, TL_DEBUG_POSITION, key)) page = table[key / a.page_size];
@@ -169,8 +172,8 @@ latent_attention_mma_kernel(const Args a) {
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int key = key0 + cw * KW + i * 8 + t4 * 2 + j;
-        s[i][j] = (on_lo && key <= pos_lo) ? s[i][j] * a.scale : -INFINITY;
-        s[i][2 + j] = (on_hi && key <= pos_hi) ? s[i][2 + j] * a.scale : -INFINITY;
+        s[i][j] = (on_lo && key <= pos_lo && key >= from_lo) ? s[i][j] * a.scale : -INFINITY;
+        s[i][2 + j] = (on_hi && key <= pos_hi && key >= from_hi) ? s[i][2 + j] * a.scale : -INFINITY;
         mx_lo = fmaxf(mx_lo, s[i][j]);
         mx_hi = fmaxf(mx_hi, s[i][2 + j]);
       }
@@ -348,7 +351,7 @@ int tl_latent_attention_mma_supported(int dk, int dv) {
 int tl_latent_attention_mma(const void* q, const void* pages, const int* block_table, int table_width,
                             const int* req_indptr, const int* kv_before, const int* tile_req, const int* tile_row,
                             int tiles, void* out, int tokens, int heads, int dk, int dv, int page_size, float scale,
-                            int num_pages, int splits, float* part_o, float* part_ml, cudaStream_t stream) {
+                            int num_pages, int splits, float* part_o, float* part_ml, int window, cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (!tl_latent_attention_mma_supported(dk, dv) || splits < 1 || splits > MAX_SPLITS) return TL_ERR_UNSUPPORTED;
   if (splits > 1 && (!part_o || !part_ml || tile_req)) return TL_ERR_UNSUPPORTED;
@@ -372,6 +375,7 @@ int tl_latent_attention_mma(const void* q, const void* pages, const int* block_t
   a.tiles_per_req = (heads + ROWS - 1) / ROWS;
   a.splits = splits;
   a.scale = scale;
+  a.window = window;
   const int ncw = dv <= 128 ? 1 : (dv <= 256 ? 2 : 4);
   const size_t smem = smem_bytes(dk, ncw);
   dim3 grid(tiles, splits);

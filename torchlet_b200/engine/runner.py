@@ -58,6 +58,30 @@ class PendingSum:
     acc: torch.Tensor
 
 
+@dataclass
+class PendingResidual:
+    """The end of a sub-layer that is left to the next norm of the stream ``acc``:
+    acc += m * norm(y (+ split sums, bias), gated) (+ row); see ``ops.residual_norm``."""
+
+    acc: torch.Tensor
+    y: torch.Tensor
+    terms: tuple  # (weight, bias or None, eps, centre) of the norm
+    m: float
+    clear: bool
+    pending: Optional[PendingSum]
+    gate: Optional[tuple]  # (float32 rows or split sums, splits or 0, bias or None)
+    row: Optional[torch.Tensor] = None
+
+    def finish(self, following=None) -> None:
+        """``following``: (weight, bias, eps, centre, out) of the norm that comes next."""
+        weight, bias, eps, centre = self.terms
+        sums, (gate, gate_splits, gate_bias) = self.pending, self.gate or (None, 0, None)
+        ops.residual_norm(self.acc, self.y, weight, eps, bias=bias, centre=centre, m=self.m,
+                          partials=sums.partials if sums else None, splits=sums.splits if sums else 0,
+                          y_bias=sums.bias if sums else None, gate=gate, gate_splits=gate_splits, gate_bias=gate_bias,
+                          row=self.row, clear=self.clear, following=following)
+
+
 class StepContext:
     """Everything a part may read about the current step."""
 
@@ -79,6 +103,7 @@ class StepContext:
         self.plans: dict = {}  # per-step plans parts share across layers
         self._pending: Optional[PendingSum] = None  # see ``leave_pending``
         self._pending_write: Optional[tuple] = None  # see ``leave_write``
+        self._residual: Optional[PendingResidual] = None  # see ``leave_residual``
         # sampling rows of the step (device), None when every sampled row is greedy
         self.num_sampled = 0
         self.sample_temperature = self.sample_seed = self.sample_counter = None
@@ -114,9 +139,38 @@ class StepContext:
         self._pending_write = None
         return pending[1:]
 
+    # A block with a norm BEHIND its sub-layers leaves that norm and the residual sum to the next norm of the stream,
+    # which does both and itself in one pass.
+    def leave_residual(self, acc, y, terms, m, clear, pending=None, gate=None) -> None:
+        self.flush_pending()
+        self._residual = PendingResidual(acc, y, terms, m, clear, pending, gate)
+        if pending is not None:
+            ops.workspace_holder = self  # its split sums still lie in the shared workspace
+
+    def take_residual(self, acc) -> Optional[PendingResidual]:
+        """The end of a sub-layer that ``acc`` still lacks, if there is one; the caller finishes it."""
+        residual = self._residual
+        if residual is None or residual.acc is not acc:
+            return None
+        self._residual = None
+        if residual.pending is not None:
+            ops.workspace_holder = None
+        return residual
+
+    def add_row(self, acc, row) -> None:
+        """acc[t] += row for every token (float32), in the kernel of a residual that is left unfinished if there is one."""
+        residual = self._residual
+        if residual is not None and residual.acc is acc and residual.row is None:
+            residual.row = row
+            return
+        self.flush_pending()
+        ops.add_row(acc, row)
+
     def flush_pending(self) -> None:
-        """Complete an unfinished sum into a stream (see ``leave_pending``) and a write that was left
-        to the next reader (see ``leave_write``)."""
+        """Complete an unfinished sum into a stream (see ``leave_pending``), the end of a sub-layer (see
+        ``leave_residual``) and a write that was left to the next reader (see ``leave_write``)."""
+        if self._residual is not None:
+            self.take_residual(self._residual.acc).finish()
         write = self._pending_write
         if write is not None:
             self._pending_write = None

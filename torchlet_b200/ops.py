@@ -47,7 +47,7 @@ _SIGNATURES = {
     "attention_generic": {
         "tl_attention_generic": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int,
-                                 c_void_p, c_int, c_void_p],
+                                 c_void_p, c_void_p, c_int, c_void_p],
         "tl_attention_generic_debug_error": [c_void_p],
     },
     "gemm_tc": {
@@ -69,8 +69,8 @@ _SIGNATURES = {
                              c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p],
         "tl_attention_mma_ex": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                 c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_int, c_void_p, c_longlong,
-                                c_void_p, c_void_p, c_void_p],
+                                c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p,
+                                c_longlong, c_void_p, c_void_p, c_void_p],
         "tl_attention_mma_error": [],
         "tl_attention_mma_debug_error": [c_void_p],
     },
@@ -84,10 +84,10 @@ _SIGNATURES = {
     "attention_tc": {
         "tl_attention_tc": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_float,
-                            c_int, c_void_p, c_int, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p, c_longlong,
-                            c_void_p, c_void_p, c_void_p],
+                            c_int, c_void_p, c_int, c_void_p, c_longlong, c_int, c_float, c_int, c_void_p, c_void_p,
+                            c_longlong, c_void_p, c_void_p, c_void_p],
         "tl_attention_tc_merge": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
-                                  c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p],
+                                  c_longlong, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p],
         "tl_attention_tc_error": [],
         "tl_attention_tc_rows": [c_int],
     },
@@ -127,7 +127,7 @@ _SIGNATURES = {
         "tl_latent_absorb_q": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                c_int, c_int, c_int, c_int, c_int, c_void_p],
         "tl_latent_attention": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+                                c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
         "tl_latent_expand_o": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
         "tl_latent_attention_debug_error": [c_void_p],
     },
@@ -135,22 +135,23 @@ _SIGNATURES = {
         "tl_latent_attention_mma_supported": [c_int, c_int],
         "tl_latent_attention_mma": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
-                                    c_void_p, c_void_p],
+                                    c_void_p, c_int, c_void_p],
         "tl_latent_attention_mma_debug_error": [c_void_p],
     },
     "gla": {
         "tl_gla_decay": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
         "tl_gla_scan": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                        c_int, c_int, c_float, c_int, c_void_p],
+                        c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_longlong, c_void_p],
         "tl_rotate_heads_f32": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-        "tl_gla_finish": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+        "tl_gla_finish": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float,
                           c_void_p],
         "tl_gla_debug_error": [c_void_p],
     },
     "gated_attention": {
         "tl_normed_qk_store": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p,
                                c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                               c_int, c_int, c_int, c_int, c_int, c_void_p],
+                               c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+        "tl_head_finish": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "tl_gated_attention_debug_error": [c_void_p],
     },
     "moe": {
@@ -175,6 +176,18 @@ _SIGNATURES = {
         "tl_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "tl_token_gate": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "tl_ssm_debug_error": [c_void_p],
+    },
+    "residual": {
+        "tl_residual_norm": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                             c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_int, c_int,
+                             c_int, c_int, c_void_p],
+        "tl_add_row": [c_void_p, c_void_p, c_int, c_int, c_void_p],
+        "tl_relu_squared": [c_void_p, c_int, c_longlong, c_void_p],
+    },
+    "token_shift": {
+        "tl_token_shift": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
+                           c_void_p, c_int, c_int, c_int, c_void_p],
+        "tl_token_shift_debug_error": [c_void_p],
     },
     "hyper": {
         "tl_hyper_fanout": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -334,11 +347,20 @@ def gemm_simt(x, w, out, bias=None, accumulate=False) -> None:
     _check(code, "gemm_simt")
 
 
+def _sink(sink, nh: int) -> tuple:
+    """(flag, address of the heads' scores or 0) of a softmax sink: False, True (score 0), or a tensor of one score a head."""
+    if not isinstance(sink, torch.Tensor):
+        return (1 if sink else 0), 0
+    _need_cuda(sink)
+    assert sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh
+    return 1, sink.data_ptr()
+
+
 def attention_generic(q, q_stride, pages, block_table, token_req, positions, out, tokens, nh, nkv, d,
-                      page_size, window, scale, softcap=None, sink: bool = False, gate=None) -> None:
+                      page_size, window, scale, softcap=None, sink=False, gate=None) -> None:
     """Paged causal GQA attention, one warp per (token, head); q may be a view into qkv.
     ``softcap``: scores become softcap * tanh(score / softcap); ``sink``: one is added to the softmax's
-    denominator; ``gate`` (float32 [tokens, >= nh * d] rows): the output is multiplied by sigmoid(gate)."""
+    denominator (True), or exp(sink[head]) (a float32 tensor [nh]); ``gate`` (float32 [tokens, >= nh * d] rows): the output is multiplied by sigmoid(gate)."""
     _need_cuda(q, pages, block_table, token_req, positions, out, gate)
     assert q.dtype == pages.dtype == out.dtype and out.is_contiguous()
     assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
@@ -346,7 +368,7 @@ def attention_generic(q, q_stride, pages, block_table, token_req, positions, out
         q.data_ptr(), q_stride, pages.data_ptr(), dtype_code(q.dtype), block_table.data_ptr(),
         block_table.shape[1], token_req.data_ptr(), positions.data_ptr(), out.data_ptr(), out.stride(0),
         tokens, nh, nkv, d, page_size, int(window or 0), float(scale), pages.shape[0], float(softcap or 0.0),
-        1 if sink else 0, _ptr(gate), gate.stride(0) if gate is not None else 0, _stream())
+        *_sink(sink, nh), _ptr(gate), gate.stride(0) if gate is not None else 0, _stream())
     _check(code, "attention_generic")
 
 
@@ -489,7 +511,8 @@ def delta_finish(o, proj, weight, out, heads: int, dim: int, eps: float) -> None
 # ----------------------------------------------------- gated linear attention
 def gla_decay(proj, low_offset: int, w2t, bias, decay, rank: int, tau: float) -> None:
     """decay[t, c] = sigmoid(z)^(1 / tau), z = W2 proj[t, low_offset : low_offset + rank] + bias, float32
-    (csrc/gla.cu).  ``w2t`` is W2 TRANSPOSED, [rank, channels]."""
+    (csrc/gla.cu); with ``tau`` 0 decay = exp(-exp(z)), z = W2 tanh(proj[...]) + bias.  ``w2t`` is W2 TRANSPOSED,
+    [rank, channels]."""
     _need_cuda(proj, w2t, bias, decay)
     tokens, channels = decay.shape
     assert proj.dtype == w2t.dtype == bias.dtype == decay.dtype == torch.float32 and proj.stride(1) == 1
@@ -500,14 +523,19 @@ def gla_decay(proj, low_offset: int, w2t, bias, decay, rank: int, tau: float) ->
 
 
 def gla_scan(proj, decay, req_indptr, slots, state, out, requests: int, heads: int, dim: int, vdim: int,
-             qscale: float, fixed_decay: bool = False, token_decay: bool = False, qk_heads: int | None = None) -> None:
+             qscale: float, fixed_decay: bool = False, token_decay: bool = False, qk_heads: int | None = None,
+             bonus=None, k_offset: int | None = None, v_offset: int | None = None) -> None:
     """Walks each request's tokens of the step through its slot's state [H, D, V] (float32):
     S = diag(decay) S + k v^T, out = S^T q * qscale; ``proj`` rows are [q (G D) | k (G D) | v (H V) | ...] with
     G = ``qk_heads`` (default H) heads of q and k, head h reading q/k head h // (H / G).
     ``decay`` is float32 [tokens, H D] (one number a key channel), or with ``fixed_decay`` one constant per head, [H]
-    (a retention), or with ``token_decay`` [tokens, H] (one number a token and head).
+    (a retention), or with ``token_decay`` [tokens, H] (one number a token and head).  ``bonus`` (float32 [H, D], a decay
+    per key channel only): out = (S_old + diag(bonus) k v^T)^T q instead.  ``k_offset``, ``v_offset``: where k and v stand
+    behind q, in numbers (default: the row layout above), so that the three may lie in planes of their own.
     A request whose slot is negative is padding."""
-    _need_cuda(proj, decay, req_indptr, slots, state, out)
+    _need_cuda(proj, decay, req_indptr, slots, state, out, bonus)
+    assert bonus is None or (bonus.dtype == torch.float32 and bonus.is_contiguous() and bonus.numel() == heads * dim
+                             and not fixed_decay and not token_decay)
     assert proj.dtype == decay.dtype == state.dtype == out.dtype == torch.float32
     assert not (fixed_decay and token_decay)
     qk_heads = heads if qk_heads is None else int(qk_heads)
@@ -516,8 +544,9 @@ def gla_scan(proj, decay, req_indptr, slots, state, out, requests: int, heads: i
     assert state.shape[1:] == (heads, dim, vdim) and req_indptr.dtype == slots.dtype == torch.int32
     code = _fn("gla", "tl_gla_scan")(proj.data_ptr(), proj.stride(0), decay.data_ptr(), req_indptr.data_ptr(),
                                      slots.data_ptr(), state.data_ptr(), out.data_ptr(), requests, heads, qk_heads, dim,
-                                     vdim, state.shape[0], float(qscale), 1 if fixed_decay else (2 if token_decay else 0),
-                                     _stream())
+                                     vdim, state.shape[0], float(qscale), 1 if fixed_decay else (2 if token_decay else (3 if bonus is not None else 0)),
+                                     _ptr(bonus), qk_heads * dim if k_offset is None else int(k_offset),
+                                     2 * qk_heads * dim if v_offset is None else int(v_offset), _stream())
     _check(code, "gla_scan")
 
 
@@ -534,25 +563,28 @@ def rotate_heads_f32(rows, positions, inv_freq, heads: int, dim: int, dims: int)
 
 def gla_finish(o, proj, gate_offset: int, weight, out, heads: int, vdim: int, eps: float) -> None:
     """out = o / rms(o per head) * weight * silu(g), g = proj[:, gate_offset:]; ``weight`` covers one head
-    (None: no weight)."""
+    [vdim] or all of them [heads vdim] (None: no weight)."""
     _need_cuda(o, proj, weight, out)
     tokens = o.shape[0]
     assert o.dtype == proj.dtype == torch.float32 and o.is_contiguous() and out.is_contiguous()
     assert out.shape == o.shape == (tokens, heads * vdim)
-    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == vdim)
-    code = _fn("gla", "tl_gla_finish")(o.data_ptr(), proj.data_ptr(), proj.stride(0), gate_offset, _ptr(weight),
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() in (vdim, heads * vdim))
+    stride = vdim if weight is not None and weight.numel() != vdim else 0
+    code = _fn("gla", "tl_gla_finish")(o.data_ptr(), proj.data_ptr(), proj.stride(0), gate_offset, _ptr(weight), stride,
                                        out.data_ptr(), dtype_code(out.dtype), tokens, heads, vdim, float(eps), _stream())
     _check(code, "gla_finish")
 
 
 # ------------------------------------------- attention with normed queries and keys
 def normed_qk_store(proj, wq, wk, inv_freq, magnitude: float, eps: float, positions, token_req, block_table, pages,
-                    page_size: int, q_out, nh: int, nkv: int, d: int, dims: int, v_offset: int, write_kv: bool = True) -> None:
+                    page_size: int, q_out, nh: int, nkv: int, d: int, dims: int, v_offset: int, write_kv: bool = True,
+                    v_inv_freq=None) -> None:
     """From float32 projection rows [q (nh d) | k (nkv d) | ...]: RMS norm of the whole q and the whole k
     (weights ``wq``, ``wk``; None: no norm), rotation of the first ``dims`` entries of every head, q to
     ``q_out``, the key to plane 0 and proj[:, v_offset : v_offset + nkv d] to plane 1 of the cache rows
-    (csrc/gated_attention.cu)."""
-    _need_cuda(proj, wq, wk, inv_freq, positions, token_req, block_table, pages, q_out)
+    (csrc/gated_attention.cu).  ``v_inv_freq`` (float32 [n]): the first 2 n entries of every value head turn by position
+    too, entry i with i + n."""
+    _need_cuda(proj, wq, wk, inv_freq, v_inv_freq, positions, token_req, block_table, pages, q_out)
     tokens = proj.shape[0]
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and q_out.is_contiguous() and pages.is_contiguous()
     assert q_out.shape == (tokens, nh * d) and pages.dtype == q_out.dtype
@@ -561,8 +593,24 @@ def normed_qk_store(proj, wq, wk, inv_freq, magnitude: float, eps: float, positi
         proj.data_ptr(), proj.stride(0), _ptr(wq), _ptr(wk), _ptr(inv_freq), float(magnitude), float(eps),
         positions.data_ptr(), token_req.data_ptr(), block_table.data_ptr(), block_table.shape[1], pages.data_ptr(),
         dtype_code(q_out.dtype), page_size, pages.shape[0], q_out.data_ptr(), tokens, nh, nkv, d, dims,
-        1 if wq is not None else 0, 1 if wk is not None else 0, v_offset, 1 if write_kv else 0, _stream())
+        1 if wq is not None else 0, 1 if wk is not None else 0, v_offset, 1 if write_kv else 0, _ptr(v_inv_freq),
+        v_inv_freq.numel() if v_inv_freq is not None else 0, _stream())
     _check(code, "normed_qk_store")
+
+
+def head_finish(rows, positions, v_inv_freq, gate, nh: int, d: int) -> None:
+    """In place on attention outputs [tokens, nh d]: the first 2 n entries of every head (``v_inv_freq`` float32 [n], or
+    None) turn by the OPPOSITE of the token's angle, entry i with i + n, and the head is multiplied by
+    sigmoid(gate[token, head]) (``gate``: float32 rows of one number a head, or None)."""
+    _need_cuda(rows, positions, v_inv_freq, gate)
+    assert rows.is_contiguous() and rows.shape[1] == nh * d and positions.dtype == torch.int32
+    assert v_inv_freq is None or (v_inv_freq.dtype == torch.float32 and v_inv_freq.is_contiguous())
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] >= nh)
+    code = _fn("gated_attention", "tl_head_finish")(
+        rows.data_ptr(), dtype_code(rows.dtype), positions.data_ptr(), _ptr(v_inv_freq), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, rows.shape[0], nh, d,
+        v_inv_freq.numel() if v_inv_freq is not None else 0, _stream())
+    _check(code, "head_finish")
 
 
 # ------------------------------------------- several residual streams, input convolution, layer norm
@@ -655,6 +703,69 @@ def hyper_write(z, y, mix, b) -> None:
     assert y.shape == (tokens, width) and mix.is_contiguous() and mix.shape == (n, n) and b.numel() == n
     _check(_fn("hyper", "tl_hyper_write")(z.data_ptr(), y.data_ptr(), mix.data_ptr(), b.data_ptr(), tokens, n, width,
                                           _stream()), "hyper_write")
+
+
+# ------------------------------------------- norms behind a sub-layer, rows added to the stream
+def residual_norm(acc, y, weight, eps: float, *, bias=None, centre: bool = False, m: float = 1.0, partials=None, splits: int = 0,
+                  y_bias=None, gate=None, gate_splits: int = 0, gate_bias=None, row=None, clear: bool = False,
+                  following=None) -> None:
+    """The end of a sub-layer and the start of the next one in one pass over the rows (csrc/residual.cu), float32:
+
+        v = y (+ the ``splits`` sums [splits, T, width] of ``partials``) (+ y_bias);   v *= sigmoid(g)
+        acc += m * norm(v) (+ row);                                                     out = norm'(acc)
+
+    norm: a layer norm (``centre``) or an RMS norm with ``weight`` (and ``bias``).  ``gate``: float32 [T, width], or with
+    ``gate_splits`` > 0 that many partial sums; ``gate_bias`` joins it.  ``row`` [width]: added to every row of acc.
+    ``clear``: y is left zeroed.  ``following`` = (weight, bias or None, eps, centre, out): the norm of the updated rows."""
+    w2 = b2 = out = None
+    eps2, centre2 = 0.0, False
+    if following is not None:
+        w2, b2, eps2, centre2, out = following
+    _need_cuda(acc, y, weight, bias, partials, y_bias, gate, gate_bias, row, w2, b2, out)
+    rows, width = acc.shape
+    for t in (acc, y, weight, bias, y_bias, gate, gate_bias, row, w2, b2, partials):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    for t in (weight, bias, y_bias, gate_bias, row, w2, b2):
+        assert t is None or t.numel() == width
+    assert y.shape == acc.shape and (gate is None or gate.numel() >= max(1, gate_splits) * rows * width)
+    assert (partials is None) == (splits == 0) and (partials is None or partials.numel() >= splits * rows * width)
+    assert out is None or (out.is_contiguous() and out.shape == acc.shape)
+    code = _fn("residual", "tl_residual_norm")(
+        acc.data_ptr(), y.data_ptr(), _ptr(partials), splits, _ptr(y_bias), _ptr(gate), max(1, gate_splits), _ptr(gate_bias),
+        weight.data_ptr(), _ptr(bias), float(eps), 1 if centre else 0, float(m), _ptr(row), _ptr(out),
+        dtype_code(out.dtype) if out is not None else 0, _ptr(w2), _ptr(b2), float(eps2), 1 if centre2 else 0, rows, width,
+        1 if clear else 0, _stream())
+    _check(code, "residual_norm")
+
+
+def add_row(acc, row) -> None:
+    """acc[t] += row for every token; float32."""
+    _need_cuda(acc, row)
+    assert acc.dtype == row.dtype == torch.float32 and acc.is_contiguous() and row.is_contiguous() and row.numel() == acc.shape[1]
+    _check(_fn("residual", "tl_add_row")(acc.data_ptr(), row.data_ptr(), acc.shape[0], acc.shape[1], _stream()), "add_row")
+
+
+def relu_squared_(x) -> None:
+    """x = max(x, 0)^2, in place, in the tensor's type."""
+    _need_cuda(x)
+    assert x.is_contiguous()
+    _check(_fn("residual", "tl_relu_squared")(x.data_ptr(), dtype_code(x.dtype), x.numel(), _stream()), "relu_squared")
+
+
+def token_shift(x, mu, out, state, token_req, req_indptr, slots, requests: int) -> None:
+    """out[c, t] = x[t] + (x[t - 1] - x[t]) * mu[c] for each of the ``mu`` rows (csrc/token_shift.cu); the row before a
+    request's first token of the step is its slot's row of ``state`` [slots, width] (float32), which then takes the
+    request's last row of the step.  out [n, >= T, width] in x's type; a negative slot is padding (zeros before it)."""
+    _need_cuda(x, mu, out, state, token_req, req_indptr, slots)
+    tokens, width = x.shape
+    n = mu.shape[0]
+    assert mu.dtype == state.dtype == torch.float32 and mu.is_contiguous() and state.is_contiguous() and mu.shape[1] == width
+    assert out.dtype == x.dtype and out.is_contiguous() and out.dim() == 3 and out.shape[0] == n and out.shape[2] == width
+    assert out.shape[1] >= tokens and x.is_contiguous() and state.shape[1:] == (width,)
+    code = _fn("token_shift", "tl_token_shift")(
+        x.data_ptr(), dtype_code(x.dtype), mu.data_ptr(), n, out.data_ptr(), out.stride(0), state.data_ptr(), state.shape[0],
+        token_req.data_ptr(), req_indptr.data_ptr(), slots.data_ptr(), requests, tokens, width, _stream())
+    _check(code, "token_shift")
 
 
 # ------------------------------ attention over a window of tokens and pooled blocks of older ones
@@ -903,7 +1014,7 @@ def latent_prepare(down, q_rank, kv_rank, rot_dim, rot_dims, q_norm, kv_norm, in
     assert not write_kv or ((q_latent is None or pages.dtype == q_latent.dtype) and pages.is_contiguous())
     code = _fn("latent_attention", "tl_latent_prepare")(
         down.data_ptr(), down.stride(0), q_rank, kv_rank, rot_dim, rot_dims, _ptr(q_norm), _ptr(kv_norm),
-        inv_freq.data_ptr(), float(eps), positions.data_ptr(), token_req.data_ptr(), block_table.data_ptr(),
+        _ptr(inv_freq), float(eps), positions.data_ptr(), token_req.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], pages.data_ptr(), dtype_code(pages.dtype), page_size, pages.shape[0],
         _ptr(q_latent), 1 if write_kv else 0, tokens, _stream())
     _check(code, "latent_prepare")
@@ -922,22 +1033,23 @@ def latent_absorb_q(q, uk, inv_freq, positions, q_abs, heads, dim, rot_dim, rot_
     assert plain_out is None or (plain_out.dtype == q_abs.dtype and plain_out.is_contiguous()
                                  and plain_out.numel() == tokens * heads * dim)
     code = _fn("latent_attention", "tl_latent_absorb_q")(
-        q.data_ptr(), q.stride(0), uk.data_ptr(), dtype_code(uk.dtype), inv_freq.data_ptr(), positions.data_ptr(),
+        q.data_ptr(), q.stride(0), uk.data_ptr(), dtype_code(uk.dtype), _ptr(inv_freq), positions.data_ptr(),
         q_abs.data_ptr(), _ptr(plain_out), tokens, heads, dim, rot_dim, rot_dims, kv_rank, 1 if fold else 0, _stream())
     _check(code, "latent_absorb_q")
 
 
 def latent_attention(q_abs, pages, block_table, token_req, positions, out, tokens, heads, dk, dv, page_size,
-                     scale) -> None:
+                     scale, window=None) -> None:
     """Causal attention of every (token, head) over the cached rows of its request, in the latent
-    space: keys are whole rows (dk), values their first dv entries; one warp per (token, head)."""
+    space: keys are whole rows (dk), values their first dv entries; one warp per (token, head).  ``window``: the mask
+    code of the paged kernels (positive: that many last positions; negative: chunks; None: all)."""
     _need_cuda(q_abs, pages, block_table, token_req, positions, out)
     assert q_abs.dtype == pages.dtype == out.dtype and q_abs.is_contiguous() and out.is_contiguous()
     assert pages.is_contiguous()
     code = _fn("latent_attention", "tl_latent_attention")(
         q_abs.data_ptr(), pages.data_ptr(), dtype_code(out.dtype), block_table.data_ptr(), block_table.shape[1],
         token_req.data_ptr(), positions.data_ptr(), out.data_ptr(), tokens, heads, dk, dv, page_size, float(scale),
-        pages.shape[0], _stream())
+        pages.shape[0], int(window or 0), _stream())
     _check(code, "latent_attention")
 
 
@@ -947,11 +1059,11 @@ def latent_attention_mma_supported(dk: int, dv: int) -> bool:
 
 
 def latent_attention_mma(q_abs, pages, block_table, req_indptr, kv_before, tile_req, tile_row, tiles, out, tokens,
-                         heads, dk, dv, page_size, scale, splits: int = 1) -> None:
+                         heads, dk, dv, page_size, scale, splits: int = 1, window=None) -> None:
     """Latent-space attention on the tensor cores (csrc/latent_attention_mma.cu), bfloat16.  Row tiles
     of 64 packed (token, head) rows: ``tile_req``/``tile_row`` name each tile's request and first row,
     or are None when every request brings one token.  ``splits`` > 1 (single tokens only): that many
-    CTAs share a request's keys and a second kernel merges them."""
+    CTAs share a request's keys and a second kernel merges them.  ``window``: as in ``latent_attention``."""
     _need_cuda(q_abs, pages, block_table, req_indptr, kv_before, tile_req, tile_row, out)
     assert q_abs.dtype == pages.dtype == out.dtype == torch.bfloat16
     assert q_abs.is_contiguous() and out.is_contiguous() and pages.is_contiguous()
@@ -963,7 +1075,7 @@ def latent_attention_mma(q_abs, pages, block_table, req_indptr, kv_before, tile_
     code = _fn("latent_attention_mma", "tl_latent_attention_mma")(
         q_abs.data_ptr(), pages.data_ptr(), block_table.data_ptr(), block_table.shape[1], req_indptr.data_ptr(),
         kv_before.data_ptr(), _ptr(tile_req), _ptr(tile_row), tiles, out.data_ptr(), tokens, heads, dk, dv, page_size,
-        float(scale), pages.shape[0], splits, _ptr(part_o), _ptr(part_ml), _stream())
+        float(scale), pages.shape[0], splits, _ptr(part_o), _ptr(part_ml), int(window or 0), _stream())
     _check(code, "latent_attention_mma", 2 if splits > 1 else 1)
 
 
@@ -1014,7 +1126,7 @@ def slot_advance(command, lanes: int, max_slots: int, sampled, records) -> None:
 
 
 # ------------------------------------------------------- tensor-core products
-EPI_STORE_BF16, EPI_ACCUM_F32, EPI_SWIGLU_BF16, EPI_STORE_F32 = 0, 1, 2, 3
+EPI_STORE_BF16, EPI_ACCUM_F32, EPI_SWIGLU_BF16, EPI_STORE_F32, EPI_RELU2_BF16 = 0, 1, 2, 3, 4
 _workspaces: dict = {}
 _outgrown: list = []  # kept alive: captured CUDA graphs may still hold their addresses
 
@@ -1071,7 +1183,7 @@ def gemm_tc(x, w, out, bias=None, epilogue=EPI_STORE_BF16, cta_pairs=None) -> No
     M, K = x.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(1) == 1
-    want = torch.bfloat16 if epilogue in (EPI_STORE_BF16, EPI_SWIGLU_BF16) else torch.float32
+    want = torch.bfloat16 if epilogue in (EPI_STORE_BF16, EPI_SWIGLU_BF16, EPI_RELU2_BF16) else torch.float32
     assert out.dtype == want and out.shape == (M, N // 2 if epilogue == EPI_SWIGLU_BF16 else N)
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N)
     need, _, splits = _gemm_plan(M, N, K)
@@ -1151,18 +1263,20 @@ def gemm_tc_grouped(x, w, out, plan, glu: bool = False, limit: float = 0.0, alph
     _check(code, "gemm_tc_grouped")
 
 
-def gemm_tc_deferred(x, w):
+def gemm_tc_deferred(x, w, workspace=None):
     """The product x @ w.T left as float32 partial sums ``[splits, M, N]`` for a fused
     finishing kernel.  Returns (partials, splits), or None when the sizes run in a
-    kernel that writes its output directly (many tokens, no K splits)."""
+    kernel that writes its output directly (many tokens, no K splits).  ``workspace``: the name of
+    a workspace of its own, so that the partial sums outlive later products (until the next call with that name)."""
     _need_cuda(x, w)
-    _release_workspace()
+    if workspace is None:
+        _release_workspace()
     M, K = x.shape
     N = w.shape[0]
     need, swap, planned = _gemm_plan(M, N, K)
     if not swap and planned <= 1:
         return None
-    ws = _workspace(x.device, need)
+    ws = _workspace(x.device if workspace is None else (workspace, x.device), need)
     splits = ctypes.c_int(0)
     code = _fn("gemm_tc", "tl_gemm_tc")(
         x.data_ptr(), w.data_ptr(), None, None, 0, EPI_STORE_F32, M, N, K, x.stride(0), w.stride(0), ws.data_ptr(),
@@ -1230,7 +1344,7 @@ _merge_in_kernel = os.environ.get("TORCHLET_B200_DECODE_MERGE", "") != "kernel"
 
 def attention_mma(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_row, tiles, out, tokens, nh, nkv,
                   d, page_size, window, scale, rows16: bool, splits: int = 1, late_wait: bool = False,
-                  softcap=None, sink: bool = False, gate=None, prior=None) -> None:
+                  softcap=None, sink=False, gate=None, prior=None) -> None:
     """Tensor-core paged attention (csrc/attention_mma.cu).  ``tile_req``/``tile_row`` None:
     tile i is request i from its first packed row.  With ``splits`` > 1 every tile is a request
     that brings one token; only those tokens' rows of ``out`` are written.  ``splits`` is the
@@ -1238,8 +1352,8 @@ def attention_mma(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile
     own length warrants.  ``late_wait`` (16-row tiles): the launch just before this one on the
     stream was ``attention_tc`` for the other requests of the same step; this grid starts beside
     it and waits for it at its end instead of at its start.  ``softcap``: scores become
-    softcap * tanh(score / softcap); ``sink``: one is added to the softmax's denominator; ``gate`` (float32
-    rows [tokens, >= nh * d]): the output is multiplied by sigmoid(gate).  ``prior`` = (ml [tokens, nh, 2], acc
+    softcap * tanh(score / softcap); ``sink``: one is added to the softmax's denominator (True), or
+    exp(sink[head]) (a float32 tensor [nh]); ``gate`` (float32 rows [tokens, >= nh * d]): the output is multiplied by sigmoid(gate).  ``prior`` = (ml [tokens, nh, 2], acc
     [tokens, nh, d]), float32: a softmax state over keys the kernel does not walk (``pooled_prior``), joined with every
     row's own where the row is normalized."""
     _need_cuda(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_row, out, gate)
@@ -1259,7 +1373,7 @@ def attention_mma(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile
         out.data_ptr(), out.stride(0), tokens, nh, nkv, d, page_size, int(window or 0), float(scale),
         1 if rows16 else 0, splits,
         _ptr(ws), ws.numel() * 4 if ws is not None else 0, _ptr(arrivals), 1 if late_wait else 0,
-        float(softcap or 0.0), 1 if sink else 0, _ptr(gate), gate.stride(0) if gate is not None else 0,
+        float(softcap or 0.0), *_sink(sink, nh), _ptr(gate), gate.stride(0) if gate is not None else 0,
         _ptr(prior_ml), _ptr(prior_acc), _stream())
     _check(code, "attention_mma", 2 if splits > 1 and arrivals is None else 1)
 
@@ -1285,7 +1399,7 @@ def attention_tc_supported(d: int, group: int, page_size: int) -> bool:
 
 def attention_tc(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_row, tiles, out, nh, nkv, d,
                  page_size, window, scale, splits: int = 1, token_req=None, defer_merge: bool = False,
-                 softcap=None, sink: bool = False, gate=None, prior=None):
+                 softcap=None, sink=False, gate=None, prior=None):
     """Prompt-portion attention on tcgen05 (csrc/attention_tc.cu): tiles of packed rows
     (``tile_row`` multiples of ``attention_tc_rows(nh // nkv)``) that cover every request of the
     step with more than one token.  ``splits`` > 1: that many CTAs share the key tiles of each
@@ -1308,7 +1422,7 @@ def attention_tc(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_
         qkv.data_ptr(), qkv.stride(0), pages.data_ptr(), pages.shape[0], block_table.data_ptr(),
         block_table.shape[1], req_indptr.data_ptr(), kv_before.data_ptr(), tile_req.data_ptr(), tile_row.data_ptr(),
         tiles, out.data_ptr(), out.stride(0), nh, nkv, d, page_size, int(window or 0), float(scale), splits,
-        _ptr(token_req), tokens, _ptr(ws), ws_bytes, 1 if defer else 0, float(softcap or 0.0), 1 if sink else 0,
+        _ptr(token_req), tokens, _ptr(ws), ws_bytes, 1 if defer else 0, float(softcap or 0.0), *_sink(sink, nh),
         _ptr(gate), gate_stride, _ptr(prior_ml), _ptr(prior_acc), _stream())
     _check(code, "attention_tc", 2 if splits > 1 and not defer else 1)
     if not defer:
@@ -1317,7 +1431,7 @@ def attention_tc(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_
     def merge() -> None:
         code = _fn("attention_tc", "tl_attention_tc_merge")(
             req_indptr.data_ptr(), out.data_ptr(), out.stride(0), nh, d, splits, token_req.data_ptr(), tokens,
-            ws.data_ptr(), ws_bytes, 1 if sink else 0, _ptr(gate), gate_stride, _ptr(prior_ml), _ptr(prior_acc),
+            ws.data_ptr(), ws_bytes, *_sink(sink, nh), _ptr(gate), gate_stride, _ptr(prior_ml), _ptr(prior_acc),
             _stream())
         _check(code, "attention_tc_merge", 1)
 
@@ -1350,7 +1464,7 @@ def debug_errors() -> list:
     found = []
     for library in ("elementwise", "attention_generic", "attention_mma", "decode_fused", "slots", "stream_ops",
                     "delta_rule", "latent_attention", "latent_attention_mma", "gla", "gated_attention", "hyper",
-                    "pooled_attention", "ssm"):
+                    "pooled_attention", "ssm", "token_shift"):
         if any(name in _functions for name in _SIGNATURES[library]):
             value = ctypes.c_int(0)
             code = _fn(library, f"tl_{library}_debug_error")(ctypes.byref(value))

@@ -126,7 +126,7 @@ def forward(mixer, ctx, qkv, cache, out, gate=None, prior=None) -> bool:
     group = nh // nkv
     if d not in (64, 128) or group > 16 or qkv.stride(0) % 8:
         return False
-    softcap, sink = getattr(mixer, "softcap", None), bool(getattr(mixer, "sink", False))
+    softcap, sink = getattr(mixer, "softcap", None), getattr(mixer, "sink", False)
     # prompt portions: the tcgen05 kernel where it takes the page size, else the mma.sync kernel
     use_tc = (not ctx.decode_only) and ops.attention_tc_supported(d, group, cache.page_size)
     plan = _plan(ctx, group, ops.attention_tc_rows(group) if use_tc else ROWS)

@@ -92,20 +92,39 @@ class Norm(Part):
     fuses_pending = False
 
     def apply(self, ctx, acc, out=None, rows=None, name="normed"):
+        if rows is None and self.residual_terms() is not None:
+            residual = ctx.take_residual(acc)
+            if residual is not None:  # the end of the sub-layer before and this norm as one kernel
+                if out is None:
+                    out = ctx.buffer(name, tuple(acc.shape), ctx.dtype)
+                residual.finish(self.residual_terms() + (out,))
+                return out
         if not self.fuses_pending:
             ctx.flush_pending()
         return self.forward(ctx, acc, out=out, rows=rows, name=name)
+
+    def residual_terms(self):
+        """(weight, bias or None, eps, centre) of a norm over whole rows that may join the end of the sub-layer before it
+        in one kernel (``ops.residual_norm``); None: not such a norm."""
+        return None
 
     def forward(self, ctx, acc, out=None, rows=None, name="normed"):
         """Return the normed ``acc`` rows (all, or those ``rows`` names, int32) in the compute
         dtype; ``out`` or a buffer called ``name`` receives them."""
         raise NotImplementedError
 
-    def add_normed(self, ctx, y, acc, m: float = 1.0, clear: bool = False) -> None:
+    def add_normed(self, ctx, y, acc, m: float = 1.0, clear: bool = False, gate=None) -> None:
         """acc += m * norm(y) in float32, for a norm that stands BEHIND a sub-layer (``y`` is the
         float32 side stream the sub-layer added its output into; ``clear``: and leave y zeroed).
-        Only norms that a block arrangement uses in that place implement it."""
-        raise NotImplementedError(f"the norm {self.kind!r} cannot stand behind a sub-layer")
+        ``gate`` = (float32 rows or split sums of them, splits or 0, bias or None): y is multiplied by
+        sigmoid(gate) first.  The sum may be left to the next norm of ``acc`` (``ctx.leave_residual``)."""
+        terms = self.residual_terms()
+        if terms is None:
+            raise NotImplementedError(f"the norm {self.kind!r} cannot stand behind a sub-layer")
+        pending = ctx.take_pending(y)
+        if pending is None:
+            ctx.flush_pending()
+        ctx.leave_residual(acc, y, terms, m, clear, pending, gate)
 
 
 class Positions(Part):

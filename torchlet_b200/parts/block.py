@@ -6,12 +6,15 @@ float32; mixer and feed-forward add into it.
 
 "parallel_scaled": one norm, mixer and feed-forward side by side, a residual multiplier.
 
-"sandwich": a norm before and behind each sub-layer: x += norm_b(f(norm_a(x))).
+"sandwich": a norm before and behind each sub-layer: x += norm_b(f(norm_a(x))), or with a gate on each sub-layer's
+result, x += norm_b(f(h) * sigmoid(W h + b)), h = norm_a(x).
 
 "hyper_connected": several residual streams a token, read and written through small learned vectors
 and a matrix per sub-layer, with an optional causal convolution over time in front of each sub-layer.
 """
 from __future__ import annotations
+
+import torch
 
 from .. import ops
 from .base import BLOCKS, Block
@@ -59,9 +62,16 @@ class SandwichBlock(Block):
     Each sub-layer adds its output into a zeroed float32 stream of its own, the norm behind it
     reads that stream and adds the normed rows into the residual stream (``Norm.add_normed``), so
     the sub-layer's output, its norm and the residual sum are all float32.  That norm's kernel also
-    leaves the side stream zeroed again, so it is cleared by a kernel of its own once a step only."""
+    leaves the side stream zeroed again, so it is cleared by a kernel of its own once a step only.
+
+    Parameter ``gates``: the names of the two sub-layers' gate matrices below the layer's prefix ([width, width], the bias
+    is the name + ``gate_bias_suffix``, default ".b").  A sub-layer's result is then multiplied, element by element, by
+    sigmoid(W h + b), h being the sub-layer's own input, before the norm behind it.  The gate's product leaves its split
+    sums (few tokens) or its float32 rows to that norm's kernel, which takes the gate, the norm, the residual sum and the
+    next sub-layer's norm in one pass."""
 
     norm_roles = ("mixer_norm", "mixer_post_norm")
+    SUBLAYERS = ("mixer", "feed_forward")
 
     def __init__(self, mixer, feed_forward, norms, params=None, token_input=None):
         super().__init__(mixer, feed_forward, norms, params, token_input)
@@ -69,6 +79,45 @@ class SandwichBlock(Block):
             missing = [role for role in ("feed_forward_norm", "feed_forward_post_norm") if role not in norms]
             if missing:
                 raise ValueError(f"block arrangement {self.kind!r} with a feed-forward needs norms for the roles {missing}")
+        self.gates = {}
+
+    @classmethod
+    def _gate_names(cls, layer) -> list:
+        """(sub-layer, full name of its gate matrix, full name of its bias) of the gates the layer has."""
+        names = layer.block_params.get("gates")
+        if not names:
+            return []
+        suffix = layer.block_params.get("gate_bias_suffix", ".b")
+        both = [(which, layer.prefix + name, layer.prefix + name + suffix) for which, name in zip(cls.SUBLAYERS, names)]
+        return both if layer.feed_forward is not None else both[:1]
+
+    @classmethod
+    def expected_tensors(cls, layer) -> list:
+        from .base import TensorSpec
+
+        out = []
+        for _, weight, bias in cls._gate_names(layer):
+            width = int(layer.norm("mixer_norm").part.params["size"])
+            out += [TensorSpec(weight, (width, width)), TensorSpec(bias, (width,), init="zeros")]
+        return out
+
+    def load(self, tensors: dict, layer, device, dtype) -> None:
+        from .linear import Linear
+
+        for which, weight, bias in self._gate_names(layer):
+            self.gates[which] = Linear(tensors[weight], tensors[bias], device, dtype)
+
+    def _gate(self, ctx, which: str, x):
+        """What ``Norm.add_normed`` takes as the gate of a sub-layer whose input is ``x`` (None: the layer has none)."""
+        linear = self.gates.get(which)
+        if linear is None:
+            return None
+        sums = linear.deferred(ctx, x, workspace="sandwich.gate")
+        if sums is not None:
+            return sums[0], sums[1], linear.bias
+        rows = ctx.buffer("sandwich.gate", (x.shape[0], linear.out_features), torch.float32)
+        linear.forward(x, rows)
+        return rows, 0, None
 
     def forward(self, ctx, acc, cache) -> None:
         side = ctx.buffer("sandwich.side", tuple(acc.shape), acc.dtype)
@@ -76,12 +125,14 @@ class SandwichBlock(Block):
         if ctx.plans.get("sandwich.side.clean") != side.data_ptr():  # the first sandwich block of the step
             ops.fill_zero(side)
             ctx.plans["sandwich.side.clean"] = side.data_ptr()
+        gate = self._gate(ctx, "mixer", x)
         self.mixer.forward(ctx, x, side, cache)
-        self.norms["mixer_post_norm"].add_normed(ctx, side, acc, clear=True)
+        self.norms["mixer_post_norm"].add_normed(ctx, side, acc, clear=True, **({"gate": gate} if gate else {}))
         if self.feed_forward is not None:
             x = self.norms["feed_forward_norm"].apply(ctx, acc)
+            gate = self._gate(ctx, "feed_forward", x)
             self.feed_forward.forward(ctx, x, side)
-            self.norms["feed_forward_post_norm"].add_normed(ctx, side, acc, clear=True)
+            self.norms["feed_forward_post_norm"].add_normed(ctx, side, acc, clear=True, **({"gate": gate} if gate else {}))
 
 
 @BLOCKS.register("hyper_connected")
@@ -150,8 +201,6 @@ class HyperConnectedBlock(Block):
         return out
 
     def load(self, tensors: dict, layer, device, dtype) -> None:
-        import torch
-
         f32 = lambda name: tensors[name].to(device=device, dtype=torch.float32).contiguous()
         for which, connection, convolution in self._names(layer):
             p = layer.prefix + connection
@@ -167,8 +216,6 @@ class HyperConnectedBlock(Block):
         return {name: StateSpec((self.taps - 1, self.width), "float32") for name in which}
 
     def _sublayer(self, ctx, z, cache, which: str, norm, run) -> None:
-        import torch
-
         tokens, n, width = z.shape
         conv = self.conv[which]
         write = ctx.take_write(z)  # the write of the sub-layer before, if it was left to us

@@ -10,9 +10,12 @@
 * ``chunk``: a query at position i sees the keys j <= i of its own chunk, floor(j / chunk) = floor(i / chunk), chunks
   counted from position 0 of the sequence (not together with ``window``);
 * ``v_dim``: the value size of a head where it differs from the key size (default ``head_dim``);
-* ``sink``: one is added to the softmax's denominator, p_j = exp(s_j) / (1 + sum exp(s_j));
+* ``sink``: one is added to the softmax's denominator, p_j = exp(s_j) / (1 + sum exp(s_j)); "learned": exp(sink_h) is,
+  one number a query head (tensor ``sink`` [H]), not scaled;
 * ``gate`` "sigmoid": the concatenated heads are multiplied by sigmoid(W_g x) before the output
-  projection; None: no gate.
+  projection; "head_sigmoid": W_g has one row a head, whose number multiplies the whole head; None: no gate;
+* ``value_rotation``: a ``rotary_partial`` part over the value heads: the value of position j turns by j before it is
+  cached, and every head's output at position i turns back by i, so a value counts by its distance; None: values stay.
 
 Query head h reads KV head h // (heads / kv_heads).  The input products (q, k, the gate) run as ONE
 product with float32 output, because norm and rotation are float32; one kernel then norms, rotates
@@ -26,7 +29,7 @@ by its ``permutation()`` in the same pass.
 
 Parameters: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``scale``, ``eps`` and the
 options above.  Tensors below the prefix: q [H D, hidden], k [G D, hidden], (v [G V, hidden]),
-q.norm [H D], k.norm [G D], g [H V, hidden], o [hidden, H V].
+q.norm [H D], k.norm [G D], g [H V or H, hidden], sink [H], o [hidden, H V].
 """
 from __future__ import annotations
 
@@ -63,15 +66,18 @@ class GatedAttentionMixer(Mixer):
             raise ValueError("a window and a chunked mask do not go together")
         # the mask code of the paged kernels: positive a sliding window, negative the chunk size, None neither
         self.window: Optional[int] = -self.chunk if self.chunk is not None else (int(p["window"]) if p.get("window") else None)
-        self.sink = bool(p.get("sink", False))
+        self.learned_sink = p.get("sink") == "learned"
+        self.sink = bool(p.get("sink", False))  # with "learned": the heads' scores, a tensor, from ``load`` on
         self.values_from_keys = bool(p.get("values_from_keys", False))
         self.qk_norm = p.get("qk_norm")
         self.gate = p.get("gate")
         self.eps = float(p.get("eps", 1e-6))
         if self.qk_norm not in (None, "whole"):
             raise ValueError(f"unknown qk_norm {self.qk_norm!r} (known: 'whole', None)")
-        if self.gate not in (None, "sigmoid"):
-            raise ValueError(f"unknown gate {self.gate!r} (known: 'sigmoid', None)")
+        if self.gate not in (None, "sigmoid", "head_sigmoid"):
+            raise ValueError(f"unknown gate {self.gate!r} (known: 'sigmoid', 'head_sigmoid', None)")
+        if p.get("sink", False) not in (False, True, None, "learned"):
+            raise ValueError(f"unknown sink {p['sink']!r} (known: True, False, 'learned')")
         if self.num_heads % self.num_kv_heads:
             raise ValueError("num_heads must be divisible by num_kv_heads")
         if self.head_dim > 256:
@@ -82,6 +88,12 @@ class GatedAttentionMixer(Mixer):
         self.positions = build_part(POSITIONS, p["positions"]) if p.get("positions") else None
         if self.positions is not None and not hasattr(self.positions, "inv_freq"):
             raise ValueError("this mixer rotates inside its own kernel and needs a position part with a frequency table")
+        self.value_rotation = build_part(POSITIONS, p["value_rotation"]) if p.get("value_rotation") else None
+        if self.value_rotation is not None and (
+                not hasattr(self.value_rotation, "inv_freq") or self.value_rotation.head_dim != self.v_dim
+                or getattr(self.value_rotation, "scaling", None) or self.values_from_keys):
+            raise ValueError("the values' rotation is a position part with a frequency table over the value size, without "
+                             "frequency scaling, for values with a projection of their own")
         self.q_size = self.num_heads * self.head_dim
         self.kv_size = self.num_kv_heads * self.head_dim
         self.in_proj: Linear | None = None
@@ -105,6 +117,10 @@ class GatedAttentionMixer(Mixer):
             out += [TensorSpec(prefix + "q.norm", (q_size,), init="ones"), TensorSpec(prefix + "k.norm", (kv_size,), init="ones")]
         if p.get("gate") == "sigmoid":
             out.append(TensorSpec(prefix + "g", (int(p["num_heads"]) * dv, hidden)))
+        if p.get("gate") == "head_sigmoid":
+            out.append(TensorSpec(prefix + "g", (int(p["num_heads"]), hidden)))
+        if p.get("sink") == "learned":
+            out.append(TensorSpec(prefix + "sink", (int(p["num_heads"]),), init="zeros"))
         out.append(TensorSpec(prefix + "o", (hidden, int(p["num_heads"]) * dv)))
         if p.get("positions"):
             out += POSITIONS.get(p["positions"].kind).expected_tensors(p["positions"], prefix)
@@ -112,24 +128,31 @@ class GatedAttentionMixer(Mixer):
 
     def load(self, tensors: dict, prefix: str, device, dtype) -> None:
         names = ["q", "k"] + ([] if self.values_from_keys else ["v"]) + (["g"] if self.gate else [])
+        part = self.value_rotation
+        v_order = part.permutation() if part is not None and hasattr(part, "permutation") else None
         order = self.positions.permutation() if self.positions is not None and hasattr(self.positions, "permutation") else None
         P = self.head_dim
 
-        def heads_of(name: str, size: int, permute: bool) -> torch.Tensor:
+        def heads_of(name: str, size: int, order) -> torch.Tensor:
             """The projection ``name`` with every head's ``size`` rows in the kernels' order, padded to P rows."""
             w = tensors[prefix + name]
-            if not self.padded and (order is None or not permute or order == list(range(size))):
+            if size == 1 and name == "g":  # one row a head
+                return w
+            if not self.padded and (order is None or order == list(range(size))):
                 return w
             w = w.reshape(-1, size, w.shape[1])
-            if permute and order is not None:
+            if order is not None:
                 w = w[:, order]
             if size != P:
                 w = torch.cat([w, w.new_zeros(w.shape[0], P - size, w.shape[2])], dim=1)
             return w.reshape(-1, w.shape[2])
 
-        sizes = {"q": (self.qk_dim, True), "k": (self.qk_dim, True), "v": (self.v_dim, False), "g": (self.v_dim, False)}
+        sizes = {"q": (self.qk_dim, order), "k": (self.qk_dim, order), "v": (self.v_dim, v_order),
+                 "g": (1, None) if self.gate == "head_sigmoid" else (self.v_dim, v_order)}
         self.in_proj = Linear(torch.cat([heads_of(n, *sizes[n]) for n in names], dim=0), None, device, dtype)
         w_o = tensors[prefix + "o"]
+        if v_order is not None and v_order != list(range(self.v_dim)):  # the heads' outputs come in the values' order
+            w_o = w_o.reshape(w_o.shape[0], self.num_heads, self.v_dim)[:, :, v_order].reshape(w_o.shape[0], -1)
         if self.padded:  # zero columns where the heads' outputs are padded
             w_o = w_o.reshape(w_o.shape[0], self.num_heads, self.v_dim)
             w_o = torch.cat([w_o, w_o.new_zeros(w_o.shape[0], self.num_heads, P - self.v_dim)], dim=2).reshape(w_o.shape[0], -1)
@@ -139,10 +162,14 @@ class GatedAttentionMixer(Mixer):
             self.k_norm = tensors[prefix + "k.norm"].to(device=device, dtype=torch.float32).contiguous()
         if self.positions is not None:
             self.positions.load(tensors, prefix, device, dtype)
+        if self.value_rotation is not None:
+            self.value_rotation.load(tensors, prefix, device, dtype)
+        if self.learned_sink:
+            self.sink = tensors[prefix + "sink"].to(device=device, dtype=torch.float32).contiguous()
         # where the projection rows hold the values and the gate
         self.v_offset = self.q_size if self.values_from_keys else self.q_size + self.kv_size
         self.gate_offset = self.q_size + self.kv_size * (1 if self.values_from_keys else 2)
-        self.proj_size = self.gate_offset + (self.q_size if self.gate else 0)
+        self.proj_size = self.in_proj.out_features
 
     def forward(self, ctx, x, acc, cache) -> None:
         tokens = x.shape[0]
@@ -154,9 +181,12 @@ class GatedAttentionMixer(Mixer):
             proj, self.q_norm, self.k_norm, positions.inv_freq if positions is not None else None,
             positions.magnitude if positions is not None else 1.0, self.eps, ctx.positions, ctx.token_req,
             cache.block_table, cache.pages, cache.page_size, q, self.num_heads, self.num_kv_heads, self.head_dim,
-            positions.dims if positions is not None else 0, self.v_offset, write_kv=cache.writable)
+            positions.dims if positions is not None else 0, self.v_offset, write_kv=cache.writable,
+            v_inv_freq=self.value_rotation.inv_freq if self.value_rotation is not None else None)
         out = ctx.buffer("gated_attention.out", (tokens, self.q_size), ctx.dtype)
-        gate = proj[:, self.gate_offset:] if self.gate else None
+        gate = proj[:, self.gate_offset:] if self.gate == "sigmoid" else None
+        if gate is not None and self.value_rotation is not None:
+            gate = None  # the output turns back first: the gate follows behind the attention kernel
         from . import attention_bf16
 
         # bfloat16 heads of 64 or 128: the tensor-core kernel (tiles of 16 packed rows for single tokens, of 64
@@ -165,5 +195,10 @@ class GatedAttentionMixer(Mixer):
             ops.attention_generic(q, q.stride(0), cache.pages, cache.block_table, ctx.token_req, ctx.positions, out, tokens,
                                   self.num_heads, self.num_kv_heads, self.head_dim, cache.page_size, self.window, self.scale,
                                   softcap=self.softcap, sink=self.sink, gate=gate)
+        if self.value_rotation is not None or self.gate == "head_sigmoid":
+            ops.head_finish(out, ctx.positions, self.value_rotation.inv_freq if self.value_rotation is not None else None,
+                            proj[:, self.gate_offset:] if self.gate == "head_sigmoid" else None, self.num_heads, self.head_dim)
+        if self.value_rotation is not None and self.gate == "sigmoid":
+            ops.gate_mul_(out, proj[:, self.gate_offset:self.gate_offset + self.q_size])
         if not self.o_proj.accumulate_later(ctx, out, acc):
             self.o_proj.forward(out, acc, accumulate=True)

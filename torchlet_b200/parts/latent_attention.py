@@ -11,7 +11,8 @@ the query and W_uv,h applied after the weighted sum of cached rows, so no key or
 cached token is ever expanded and prompt portions, single tokens and mixed batches are one code
 path.  A layer with ``kv_from`` has no W_dkv and reads another layer's cache rows.
 
-Options: ``q_rank`` None: there is no query latent, q = W_q x (tensor ``q`` instead of dq, dq.norm, uq);
+Options: ``rot_dim`` 0: no rotated part (no positions at all; the cache row is c alone); ``window``: a query at position i
+sees the keys j with 0 <= i - j < window only (None: all before it); ``q_rank`` None: there is no query latent, q = W_q x (tensor ``q`` instead of dq, dq.norm, uq);
 ``gate`` "sigmoid": the concatenated heads are multiplied by sigmoid(W_g x) (tensor ``g``) before W_o;
 ``pairing`` "interleaved": the checkpoint rotates entry 2i with 2i + 1; the rotated rows of W_q (or W_uq) and of W_dkv
 are then laid out at load time so that the kernels' split-half rotation turns the same pairs (q and k alike, so every
@@ -19,7 +20,7 @@ score is what it was).
 
 Parameters: ``hidden_size``, ``num_heads``, ``head_dim`` (unrotated), ``rot_dim``, ``v_dim``,
 ``q_rank``, ``kv_rank``, ``scale``, ``rot_base``, ``rot_dims`` (how many of the rot_dim entries
-are rotated), ``eps``, ``own_kv``, ``gate``, ``pairing``.  Tensors below the prefix: dq, dq.norm, uq (or q),
+are rotated), ``eps``, ``own_kv``, ``gate``, ``pairing``, ``window``.  Tensors below the prefix: dq, dq.norm, uq (or q),
 [dkv, dkv.norm], uk, uv, [g], o.
 """
 from __future__ import annotations
@@ -46,19 +47,20 @@ def _sm_count(device_index: int) -> int:
     return torch.cuda.get_device_properties(device_index).multi_processor_count
 
 
-def row_tiles(ctx, heads: int):
+def row_tiles(ctx, heads: int, window=None):
     """The row tiles of a step for the tensor-core kernel: (tile_req, tile_row, tiles, key splits),
-    planned once a step for every layer with the same number of heads.  A step of single tokens
+    planned once a step for every layer with the same number of heads and window.  A step of single tokens
     plans nothing on the host (tile i is request i's) and splits each request's keys over as many
     CTAs as fill the GPU once, given the longest request the step may meet; the kernel decides on
     the device how many key tiles a split really has."""
-    key = ("latent_attention.tiles", heads)
+    key = ("latent_attention.tiles", heads, window)
     plan = ctx.plans.get(key)
     if plan is None:
         if ctx.decode_only:
             tiles = ctx.num_requests * (-(-heads // ROWS))
             room = max(1, 2 * _sm_count(torch.cuda.current_device()) // tiles)
-            splits = max(1, min(room, -(-ctx.max_kv_len // MIN_KEYS_A_SPLIT), 64))
+            keys = ctx.max_kv_len if window is None else min(ctx.max_kv_len, window)
+            splits = max(1, min(room, -(-keys // MIN_KEYS_A_SPLIT), 64))
             plan = (None, None, tiles, splits)
         else:
             indptr = ctx.req_indptr_host
@@ -91,8 +93,9 @@ class LatentAttentionMixer(Mixer):
         self.pairing = p.get("pairing", "split_half")
         if self.gate not in (None, "sigmoid"):
             raise ValueError(f"unknown gate {self.gate!r} (known: 'sigmoid', None)")
+        self.window = int(p["window"]) if p.get("window") else None
         self.scale = float(p["scale"])
-        self.rot_base = float(p["rot_base"])
+        self.rot_base = float(p.get("rot_base", 10000.0))
         self.rot_dims = int(p.get("rot_dims", self.rot_dim))
         self.eps = float(p["eps"])
         self.own_kv = bool(p.get("own_kv", True))
@@ -111,7 +114,7 @@ class LatentAttentionMixer(Mixer):
         self.uk = self.uv = self.uk_heads = self.q_norm = self.kv_norm = self.inv_freq = None
 
     def kv_spec(self) -> KVSpec:
-        return KVSpec(1, self.row, None, planes=1)
+        return KVSpec(1, self.row, self.window, planes=1)
 
     @classmethod
     def expected_tensors(cls, spec: PartSpec, prefix: str) -> list[TensorSpec]:
@@ -206,13 +209,13 @@ class LatentAttentionMixer(Mixer):
                                 self.rot_dims, self.kv_rank)
         o_lat = ctx.buffer("latent.o_lat", (tokens, H * self.kv_rank), ctx.dtype)
         if ctx.dtype == torch.bfloat16 and ops.latent_attention_mma_supported(self.row, self.kv_rank):
-            tile_req, tile_row, tiles, splits = row_tiles(ctx, H)
+            tile_req, tile_row, tiles, splits = row_tiles(ctx, H, self.window)
             ops.latent_attention_mma(q_abs, cache.pages, cache.block_table, ctx.req_indptr, ctx.kv_before, tile_req,
                                      tile_row, tiles, o_lat, tokens, H, self.row, self.kv_rank, cache.page_size,
-                                     self.scale, splits)
+                                     self.scale, splits, window=self.window)
         else:
             ops.latent_attention(q_abs, cache.pages, cache.block_table, ctx.token_req, ctx.positions, o_lat, tokens, H,
-                                 self.row, self.kv_rank, cache.page_size, self.scale)
+                                 self.row, self.kv_rank, cache.page_size, self.scale, window=self.window)
         out = ctx.buffer("latent.out", (tokens, H * self.v_dim), ctx.dtype)
         if per_head_products:
             V, rank = self.v_dim, self.kv_rank

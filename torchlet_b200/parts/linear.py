@@ -29,13 +29,13 @@ class Linear:
         self.weight, self.bias, self.dtype = weight, None, weight.dtype
         return self
 
-    def deferred(self, ctx, x: torch.Tensor):
+    def deferred(self, ctx, x: torch.Tensor, workspace=None):
         """For few tokens in bfloat16: run the product but leave its split partial sums
         for a fused finishing kernel.  Returns (partials, splits) or None (not applicable;
-        use ``forward``)."""
+        use ``forward``).  ``workspace``: keep them in a workspace of that name (``ops.gemm_tc_deferred``)."""
         if self.dtype != torch.bfloat16 or not ops.gemm_tc_supported(x, self.weight):
             return None
-        return ops.gemm_tc_deferred(x, self.weight)
+        return ops.gemm_tc_deferred(x, self.weight, workspace)
 
     def accumulate_later(self, ctx, x: torch.Tensor, acc: torch.Tensor) -> bool:
         """acc += x W^T + b, with the final sum left to whoever reads ``acc`` next

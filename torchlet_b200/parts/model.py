@@ -41,6 +41,8 @@ def _layer_parts(layer) -> list:
 def expected_tensors(spec: ModelSpec) -> list[TensorSpec]:
     """Every tensor the checkpoint must hold, by name, with its shape."""
     out = [TensorSpec(spec.embedding_name, (spec.vocab_size, spec.hidden_size))]
+    if spec.stream_rows_name is not None:
+        out.append(TensorSpec(spec.stream_rows_name, (spec.stream_rows, spec.hidden_size)))
     if spec.embedding_norm is not None:
         out += NORMS.get(spec.embedding_norm.kind).expected_tensors(spec.embedding_norm, spec.embedding_norm_prefix)
     for layer in spec.layers:
@@ -79,6 +81,7 @@ class LayeredModel:
         self.final_norm = build_part(NORMS, spec.final_norm)
         self.embedding_norm = build_part(NORMS, spec.embedding_norm) if spec.embedding_norm is not None else None
         self.embedding: torch.Tensor | None = None
+        self.stream_rows: torch.Tensor | None = None  # [rows, hidden] float32, see ``ScheduleEntry.add_row``
         self.lm_head: Linear | None = None
         self.dtype: torch.dtype | None = None
         self.device = None
@@ -104,6 +107,8 @@ class LayeredModel:
         spec = self.spec
         self.device, self.dtype = torch.device(device), dtype
         self.embedding = tensors[spec.embedding_name].to(device=device, dtype=dtype).contiguous()
+        if spec.stream_rows_name is not None:
+            self.stream_rows = tensors[spec.stream_rows_name].to(device=device, dtype=torch.float32).contiguous()
         for layer, block in zip(spec.layers, self.blocks):
             for _, _, prefix, role in _layer_parts(layer):
                 part = {"mixer": block.mixer, "feed_forward": block.feed_forward,
@@ -141,6 +146,8 @@ class LayeredModel:
                 if entry.add_embedding:
                     ctx.flush_pending()
                     ops.scaled_add(acc, first, 1.0)
+                if entry.add_row is not None:
+                    ctx.add_row(acc, self.stream_rows[entry.add_row])
                 self.blocks[entry.layer].forward(ctx, acc, caches[i])
             ctx.flush_pending()
             return acc

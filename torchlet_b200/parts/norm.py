@@ -59,11 +59,17 @@ class RMSNorm(Norm):
         ops.rms_norm(acc, self.weight, self.eps, out, rows, self.groups)
         return out
 
-    def add_normed(self, ctx, y, acc, m: float = 1.0, clear: bool = False) -> None:
+    def residual_terms(self):
+        return (self.weight, None, self.eps, False) if self.groups == 1 else None
+
+    def add_normed(self, ctx, y, acc, m: float = 1.0, clear: bool = False, gate=None) -> None:
         """acc += m * norm(y): both float32 ``[T, size]``; ``y`` is a side stream a sub-layer added its
         output into.  ``clear``: y is zeroed in the same pass, ready for the next sub-layer."""
         if self.groups != 1:
             raise ValueError("the norm of a sub-layer's output is not built for grouped norms")
+        if gate is not None:
+            super().add_normed(ctx, y, acc, m, clear, gate)
+            return
         pending = ctx.take_pending(y)
         if pending is not None and pending.bias is None:
             # the sub-layer's last product left its split sums: their sum into y, the norm and the residual sum
@@ -84,6 +90,9 @@ class LayerNorm(Norm):
     prefix itself is the tensor's name), ``bias_name`` (default "bias"; None: no bias)."""
 
     centre = True
+
+    def residual_terms(self):
+        return self.weight, self.bias, self.eps, True
 
     def __init__(self, spec: PartSpec):
         super().__init__(spec)
