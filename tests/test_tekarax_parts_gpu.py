@@ -364,6 +364,55 @@ def test_time_mixing_products_at_many_token_counts(tokens):
     close(outs[1][1], outs[0][1].double(), 3e-2, "states")
 
 
+@pytest.mark.parametrize("H,D,rank,width", [(3, 16, 5, 64), (2, 20, 40, 72), (4, 32, 1, 64), (2, 64, 24, 128), (1, 96, 70, 64),
+                                            (3, 128, 200, 128), (2, 100, 100, 64)])
+@pytest.mark.parametrize("tokens", [1, 5, 16, 20, 40, 64])
+def test_single_tokens_in_one_kernel_walk_on_as_the_portions_do(H, D, rank, width, tokens):
+    """Many requests, one token each, four steps in a row from states that a portion has left, every third lane padding,
+    slots in a scrambled order: the stacked products and the one-kernel step against the plain recurrence."""
+    from torchlet_b200 import ops
+    from torchlet_b200.config import PartSpec
+    from torchlet_b200.parts import MIXERS, build_part
+
+    td, eps, steps = torch.bfloat16, 1e-5, 4
+    m, w = {"heads": H, "dim": D}, _mixing_weights(H, D, rank, width, seed=D)
+    part = build_part(MIXERS, PartSpec("time_mixing", {"hidden_size": width, "num_heads": H, "head_dim": D, "decay_rank": rank, "eps": eps}))
+    part.load(w, "t.", DEV, td)
+    no_deferred_sums(part)
+    assert part.one_kernel
+    slots = torch.randperm(tokens + 2, generator=torch.Generator().manual_seed(tokens))[:tokens].tolist()
+    slots = [-1 if i % 3 == 2 else s for i, s in enumerate(slots)]
+    live = [i for i, s in enumerate(slots) if s >= 0]
+    state = {name: torch.full((tokens + 2, *spec.slot_shape(64)), float("nan"), device=DEV) for name, spec in part.state_spec().items()}
+    for t in state.values():
+        for i in live:
+            t[slots[i]] = 0.0
+    seqs = {i: rand(6 + steps, width, seed=100 + i).to(td).float() for i in live}
+    for i in live:  # six tokens as a portion
+        part.forward(Ctx(td, [6], [0], [slots[i]], capacity=512), seqs[i][:6].to(td).to(DEV), torch.zeros(6, width, device=DEV), Cache(state))
+    calls, inner = [], ops.time_mixing_step
+    ops.time_mixing_step = lambda *a, **k: (calls.append(1), inner(*a, **k))
+    try:
+        got = []
+        for k in range(steps):
+            x = torch.stack([seqs[i][6 + k] if i in seqs else torch.ones(width) for i in range(tokens)])
+            acc = torch.zeros(tokens, width, device=DEV)
+            part.forward(Ctx(td, [1] * tokens, [6 + k] * tokens, slots, capacity=512), x.to(td).to(DEV), acc, Cache(state))
+            got.append(acc.cpu())
+            for i in range(tokens):
+                if slots[i] < 0:
+                    assert float(acc[i].abs().max()) == 0.0
+    finally:
+        ops.time_mixing_step = inner
+    assert len(calls) == steps
+    for i in live[:: max(1, len(live) // 6)]:
+        want = plain.wkv(m, double(w), "t.", seqs[i].double(), eps)[6:]
+        close(torch.stack([g[i] for g in got]), want, 6e-2, f"request {i}")
+    for t in state.values():  # slots nobody owns are as they were
+        owned = {slots[i] for i in live}
+        assert all(bool(torch.isnan(t[s]).all()) == (s not in owned) for s in range(tokens + 2))
+
+
 def test_the_bonus_meets_the_current_token_only_and_the_state_remembers():
     """A decay near one keeps the first token's value for 600 tokens, through portions and single tokens; the bonus shows
     in a token's own output and never in the state."""

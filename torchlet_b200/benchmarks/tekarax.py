@@ -49,7 +49,7 @@ def tekarax_config(size: str, layers: int, experts: int = 8, top: int = 2, windo
 
 
 KERNEL_CLASSES = {
-    "time mixing (shift, decay, scan, norm and gate)": ("token_shift", "gla_decay", "gla_scan", "gla_finish"),
+    "time mixing (shift, decay, scan, norm and gate)": ("token_shift", "time_mixing_step", "gla_decay", "gla_scan", "gla_finish"),
     "attention (rotations, cache write, turning back and head gates)": ("normed_qk_store", "head_finish"),
     "attention (scores and values)": ("attention_tc", "attention_mma", "attention_generic"),
     "latent attention (prepare, absorb, scores and values, expand)":

@@ -25,6 +25,45 @@ using namespace tl;
 
 constexpr int MAX_HALF = 128;  // rotated pairs of a head of up to 256 entries
 
+template <int V> __device__ __forceinline__ void load_some(const float* p, float (&v)[V]) {
+#pragma unroll
+  for (int j = 0; j < V; j += 4) {
+    if constexpr (V % 4 == 0) {
+      const float4 x = *reinterpret_cast<const float4*>(p + j);
+      v[j] = x.x; v[j + 1] = x.y; v[j + 2] = x.z; v[j + 3] = x.w;
+    } else {
+      v[j] = p[j];
+    }
+  }
+}
+template <int V> __device__ __forceinline__ void load_some(const __nv_bfloat16* p, float (&v)[V]) {
+  if constexpr (V == 8) load8(p, v);
+  else v[0] = __bfloat162float(*p);
+}
+template <int V> __device__ __forceinline__ void store_some(float* p, const float (&v)[V]) {
+#pragma unroll
+  for (int j = 0; j < V; j += 4) {
+    if constexpr (V % 4 == 0) *reinterpret_cast<float4*>(p + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+    else p[j] = v[j];
+  }
+}
+template <int V> __device__ __forceinline__ void store_some(__nv_bfloat16* p, const float (&v)[V]) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+  } else if constexpr (V == 8) {
+    uint32_t w[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+      w[j] = *reinterpret_cast<const uint32_t*>(&h);
+    }
+    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+  } else {
+    *p = __float2bfloat16_rn(v[0]);
+  }
+}
+
 // NT threads a token: 256 up to 1,024 entries of q and k together, 512 up to 4,096, 1,024 beyond, so that a thread
 // walks few entries one after the other.
 template <typename T, int NT>
@@ -113,39 +152,133 @@ normed_qk_store_kernel(const float* __restrict__ proj, int proj_stride, const fl
   }
 }
 
-template <int V> __device__ __forceinline__ void load_some(const float* p, float (&v)[V]) {
-#pragma unroll
-  for (int j = 0; j < V; j += 4) {
-    if constexpr (V % 4 == 0) {
-      const float4 x = *reinterpret_cast<const float4*>(p + j);
-      v[j] = x.x; v[j + 1] = x.y; v[j + 2] = x.z; v[j + 3] = x.w;
+// The same where every size is a multiple of 4 and everything is 16-byte aligned: a thread takes four neighbouring pairs (or
+// four entries that do not turn) of a head at a time, and has its first ones on their way before the cosines are taken.
+template <typename T, int NT>
+__global__ void __launch_bounds__(NT)
+normed_qk_store_wide_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ wq,
+                            const float* __restrict__ wk, const float* __restrict__ inv_freq, float magnitude, float eps,
+                            const int* __restrict__ positions, const int* __restrict__ token_req,
+                            const int* __restrict__ block_table, int table_width, T* __restrict__ pages, int page_size,
+                            int num_pages, T* __restrict__ q_out, int nh, int nkv, int d, int dims, int norm_q, int norm_k,
+                            int v_offset, int write_kv, const float* __restrict__ v_inv_freq, int v_half) {
+  tl::pdl_launch_dependents();
+  tl::pdl_wait();
+  __shared__ float scratch[32];
+  __shared__ __align__(16) float turn[4][MAX_HALF];
+  const int t = blockIdx.x;
+  const float* row = proj + (size_t)t * proj_stride;
+  const int qn = nh * d, kn = nkv * d, half = dims >> 1;
+  const int pos = positions[t];
+  const float p = (float)pos;
+  // items: the quads of the q heads, then of the k heads, then of the v heads
+  const int per_qk = (half >> 2) + ((d - dims) >> 2), per_v = (v_half >> 2) + ((d - 2 * v_half) >> 2);
+  const int q_items = nh * per_qk, k_items = write_kv ? nkv * per_qk : 0, v_items = write_kv ? nkv * per_v : 0;
+  const int items = q_items + k_items + v_items;
+  struct Quad {
+    int what, head, e, partner;  // 0 q, 1 k, 2 v; the entry in its head; how far the partner stands (0: it does not turn)
+  };
+  auto quad_of = [&](int item) {
+    Quad x;
+    x.what = item < q_items ? 0 : (item < q_items + k_items ? 1 : 2);
+    const int local = x.what == 0 ? item : (x.what == 1 ? item - q_items : item - q_items - k_items);
+    const int per = x.what == 2 ? per_v : per_qk, n = x.what == 2 ? v_half : half;
+    x.head = local / per;
+    const int i = local - x.head * per;
+    x.partner = i < (n >> 2) ? n : 0;
+    x.e = x.partner ? i * 4 : 2 * n + (i - (n >> 2)) * 4;
+    return x;
+  };
+  auto source = [&](const Quad& x) { return row + (x.what == 0 ? 0 : (x.what == 1 ? qn : v_offset)) + x.head * d + x.e; };
+  float a[4], b[4];
+  auto fetch = [&](const Quad& x) {
+    const float* src = source(x);
+    load_some<4>(src, a);
+    if (x.partner) load_some<4>(src + x.partner, b);
+  };
+  Quad now{};
+  if (threadIdx.x < items) {
+    now = quad_of(threadIdx.x);
+    fetch(now);
+  }
+  for (int i = threadIdx.x; i < half + v_half; i += NT) {
+    float sn, cs;
+    if (i < half) {
+      sincosf(p * inv_freq[i], &sn, &cs);
+      turn[0][i] = cs * magnitude;
+      turn[1][i] = sn * magnitude;
     } else {
-      v[j] = p[j];
+      sincosf(p * v_inv_freq[i - half], &sn, &cs);
+      turn[2][i - half] = cs;
+      turn[3][i - half] = sn;
     }
   }
-}
-template <int V> __device__ __forceinline__ void load_some(const __nv_bfloat16* p, float (&v)[V]) {
-  if constexpr (V == 8) load8(p, v);
-  else v[0] = __bfloat162float(*p);
-}
-template <int V> __device__ __forceinline__ void store_some(float* p, const float (&v)[V]) {
-#pragma unroll
-  for (int j = 0; j < V; j += 4) {
-    if constexpr (V % 4 == 0) *reinterpret_cast<float4*>(p + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
-    else p[j] = v[j];
-  }
-}
-template <int V> __device__ __forceinline__ void store_some(__nv_bfloat16* p, const float (&v)[V]) {
-  if constexpr (V == 8) {
-    uint32_t w[4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
-      w[j] = *reinterpret_cast<const uint32_t*>(&h);
+  float inv_q = 1.f, inv_k = 1.f;
+  auto mean_square = [&](const float* x, int n) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * 4; i < n; i += NT * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(x + i);
+      ss = fmaf(v.x, v.x, ss);
+      ss = fmaf(v.y, v.y, ss);
+      ss = fmaf(v.z, v.z, ss);
+      ss = fmaf(v.w, v.w, ss);
     }
-    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
-  } else {
-    *p = __float2bfloat16_rn(v[0]);
+    return block_sum<NT>(ss, scratch) / (float)n;
+  };
+  if (norm_q) inv_q = 1.f / sqrtf(mean_square(row, qn) + eps);
+  if (norm_k) inv_k = 1.f / sqrtf(mean_square(row + qn, kn) + eps);
+  __syncthreads();
+  // pages: [num_pages, 2, nkv, page_size, d]
+  T* kdst = nullptr;
+  if (write_kv) {
+    int page = -1;
+    if (TL_DEBUG_OK(pos / page_size < table_width, TL_DEBUG_POSITION, pos))
+      page = block_table[(size_t)token_req[t] * table_width + pos / page_size];
+    if (TL_DEBUG_OK(page >= 0 && page < num_pages, TL_DEBUG_PAGE, page) && page >= 0)
+      kdst = pages + (size_t)page * 2 * nkv * page_size * d + (size_t)(pos % page_size) * d;
+  }
+  for (int item = threadIdx.x; item < items;) {
+    const float inv = now.what == 0 ? inv_q : (now.what == 1 ? inv_k : 1.f);
+    const float* w = now.what == 0 ? (norm_q ? wq : nullptr) : (now.what == 1 && norm_k ? wk : nullptr);
+    const int at = now.head * d + now.e;
+    float x[4], y[4];
+    if (w) {
+      float wa[4];
+      load_some<4>(w + at, wa);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) a[j] = a[j] * inv * wa[j];
+      if (now.partner) {
+        load_some<4>(w + at + now.partner, wa);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) b[j] = b[j] * inv * wa[j];
+      }
+    }
+    if (now.partner) {
+      float cs[4], sn[4];
+      load_some<4>(&turn[now.what == 2 ? 2 : 0][now.e], cs);
+      load_some<4>(&turn[now.what == 2 ? 3 : 1][now.e], sn);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        x[j] = a[j] * cs[j] - b[j] * sn[j];
+        y[j] = b[j] * cs[j] + a[j] * sn[j];
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[j] = a[j];
+    }
+    T* dst = q_out + (size_t)t * qn + at;
+    if (now.what != 0)
+      dst = kdst ? kdst + (size_t)((now.what == 2 ? nkv : 0) + now.head) * page_size * d + now.e : nullptr;
+    const int partner = now.partner;
+    item += NT;
+    if (item < items) {
+      now = quad_of(item);
+      fetch(now);
+    }
+    if (dst) {
+      store_some<4>(dst, x);
+      if (partner) store_some<4>(dst + partner, y);
+    }
   }
 }
 
@@ -222,6 +355,22 @@ extern "C" int tl_normed_qk_store(const float* proj, int proj_stride, const floa
   if (d <= 0 || dims < 0 || dims > d || dims % 2 || nh <= 0 || nkv <= 0 || page_size <= 0) return TL_ERR_UNSUPPORTED;
   if (dims / 2 > MAX_HALF || v_half < 0 || v_half > MAX_HALF || 2 * v_half > d || (v_half && !v_inv_freq)) return TL_ERR_UNSUPPORTED;
   const long long width = (long long)(nh + nkv) * d;
+  const uintptr_t all = (uintptr_t)proj | (uintptr_t)wq | (uintptr_t)wk | (uintptr_t)pages | (uintptr_t)q_out;
+  if (d % 4 == 0 && dims % 8 == 0 && v_half % 4 == 0 && proj_stride % 4 == 0 && v_offset % 4 == 0 && (all & 15) == 0) {
+#define TL_STORE_WIDE(T, NT)                                                                                               \
+  tl::launch_kernel(normed_qk_store_wide_kernel<T, NT>, (unsigned)tokens, NT, 0, stream, proj, proj_stride, wq, wk, inv_freq, \
+                    magnitude, eps, positions, token_req, block_table, table_width, (T*)pages, page_size, num_pages,         \
+                    (T*)q_out, nh, nkv, d, dims, norm_q, norm_k, v_offset, write_kv, v_inv_freq, v_half)
+    if (dtype == TL_DTYPE_F32) {
+      if (width <= 2048) TL_STORE_WIDE(float, 128);
+      else TL_STORE_WIDE(float, 256);
+    } else {
+      if (width <= 2048) TL_STORE_WIDE(__nv_bfloat16, 128);
+      else TL_STORE_WIDE(__nv_bfloat16, 256);
+    }
+#undef TL_STORE_WIDE
+    return TL_LAUNCH_CHECK();
+  }
 #define TL_STORE(T, NT)                                                                                              \
   tl::launch_kernel(normed_qk_store_kernel<T, NT>, (unsigned)tokens, NT, 0, stream, proj, proj_stride, wq, wk, inv_freq, \
                     magnitude, eps, positions, token_req, block_table, table_width, (T*)pages, page_size, num_pages,     \

@@ -76,6 +76,10 @@ struct Params {
   // [g group_rows, (g + 1) group_rows) of the column operand.  nullptr: one group.
   const int* plan;
   int group_rows;
+  // stacked products (swapped kernel): column tile y times weight rows [y group_rows, (y + 1) group_rows) of a row operand
+  // of ``stack_rows`` rows in all (the last group may have fewer); 0: not stacked.  Known before the launch, so the weight
+  // stream starts before the wait.
+  int stack_rows;
 };
 
 __device__ __forceinline__ float silu(float g) { return g / (1.f + __expf(-g)); }
@@ -262,6 +266,9 @@ gemm_tc_swapped_kernel(const __grid_constant__ CUtensorMap map_row, const __grid
     const int group = (int)blockIdx.y < p.plan[0] ? p.plan[1 + blockIdx.y] : -1;
     if (group < 0) num_kb = 0;
     else wrow0 = group * p.group_rows + row0;
+  } else if (p.stack_rows) {
+    wrow0 = (int)blockIdx.y * p.group_rows + row0;
+    if (wrow0 >= p.stack_rows) num_kb = 0;
   }
 
   if (threadIdx.x == 0) {
@@ -1105,6 +1112,7 @@ static int gemm_tc_impl(const void* x, const void* w, const float* bias, void* o
   p.row_scale = row_scale;
   p.plan = nullptr;
   p.group_rows = 0;
+  p.stack_rows = 0;
   if (splits_out) *splits_out = 0;
   CUtensorMap map_row, map_col;
   int rc;
@@ -1219,6 +1227,54 @@ static int gemm_tc_impl(const void* x, const void* w, const float* bias, void* o
   return TL_LAUNCH_CHECK();
 }
 
+// Several products of FEW rows each as one launch: x [groups * group_cols, K] (group g's rows from g * group_cols on), w
+// [stack_rows, K] (group g's matrix in rows [g N, (g + 1) N), the last group may have fewer rows), left as float32 partial
+// sums [splits][groups * group_cols][N] in ``workspace``; *splits_out gets their number (at least 1).  Columns past a
+// short last group's rows are not written.  group_cols 16, 32 or 64.  With workspace == nullptr only *splits_out is set.
+int tl_gemm_tc_stacked(const void* x, const void* w, int groups, int group_cols, int N, int K, int stack_rows, void* workspace,
+                       long long workspace_bytes, int* splits_out, cudaStream_t stream) {
+  if (groups <= 0 || N <= 0 || K <= 0 || K % 8 || stack_rows <= (groups - 1) * N || stack_rows > groups * N) return TL_ERR_UNSUPPORTED;
+  if (group_cols != 16 && group_cols != 32 && group_cols != 64) return TL_ERR_UNSUPPORTED;
+  const int k_blocks = (K + BLOCK_K - 1) / BLOCK_K;
+  const int row_tiles = (N + BLOCK_P - 1) / BLOCK_P;
+  const int tiles = (groups - 1) * row_tiles + (stack_rows - (groups - 1) * N + BLOCK_P - 1) / BLOCK_P;
+  int splits = 2 * sm_count() / tiles;
+  if (splits < 1) splits = 1;
+  if (splits > k_blocks / 4) splits = k_blocks / 4 > 0 ? k_blocks / 4 : 1;  // at least 4 k-blocks a split
+  Params p;
+  p.k_blocks = k_blocks;
+  p.k_blocks_per_split = (k_blocks + splits - 1) / splits;
+  splits = (k_blocks + p.k_blocks_per_split - 1) / p.k_blocks_per_split;
+  if (splits_out) *splits_out = splits;
+  if (!workspace) return 0;
+  if ((long long)splits * groups * group_cols * N * 4 > workspace_bytes) return TL_ERR_UNSUPPORTED;
+  p.bias = nullptr;
+  p.out = nullptr;
+  p.ldo = 0;
+  p.epilogue = EPI_STORE_F32;
+  p.partial = (float*)workspace;
+  p.splits = 1;
+  p.ahead = 8;
+  p.glu_limit = p.glu_alpha = 0.f;
+  p.row_scale = nullptr;
+  p.plan = nullptr;
+  p.group_rows = N;
+  p.stack_rows = stack_rows;
+  p.rows = N;
+  p.cols = groups * group_cols;
+  p.block_q = group_cols;
+  p.stages = p.row_tiles = p.num_tiles = 0;
+  CUtensorMap map_row, map_col;
+  if (!cached_map(&map_row, w, stack_rows, K, K, BLOCK_P) || !cached_map(&map_col, x, (uint64_t)p.cols, K, K, group_cols))
+    return TL_ERR_UNSUPPORTED;
+  const dim3 grid(row_tiles, groups, splits);
+  switch (group_cols) {
+    case 16: return launch_swapped<16, 6>(map_row, map_col, p, grid, stream);
+    case 32: return launch_swapped<32, 4>(map_row, map_col, p, grid, stream);
+    default: return launch_swapped<64, 4>(map_row, map_col, p, grid, stream);
+  }
+}
+
 // Grouped product over group-sorted rows: x [rows, K] (rows a multiple of 128; row tile i belongs to group
 // plan[1 + i], plan[0] tiles are in use), w [groups * N, K] (group g's matrix in rows [g N, (g + 1) N)),
 // out [rows, N] (or [rows, N / 2] with the gated epilogue over 16-interleaved gate / up rows).  The plan is
@@ -1250,6 +1306,7 @@ int tl_gemm_tc_grouped(const void* x, const void* w, void* out, long long ldo, i
     p.row_scale = nullptr;
     p.plan = plan;
     p.group_rows = N;
+    p.stack_rows = 0;
     p.rows = N;     // weight rows of one group
     p.cols = rows;  // sorted rows
     p.block_q = 16;
@@ -1276,6 +1333,7 @@ int tl_gemm_tc_grouped(const void* x, const void* w, void* out, long long ldo, i
   p.row_scale = nullptr;
   p.plan = plan;
   p.group_rows = N;
+  p.stack_rows = 0;
   p.rows = rows;
   p.cols = N;
   int block_q = 256;

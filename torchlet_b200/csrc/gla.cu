@@ -41,12 +41,13 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
                  float inv_tau) {  // inv_tau > 0: sigmoid(z)^(inv_tau); 0: exp(-exp(z)) of a tanh of the low-rank input
   tl::pdl_launch_dependents();
   tl::pdl_wait();
-  extern __shared__ float low[];  // DECAY_TOKENS x rank
+  extern __shared__ __align__(16) float low[];  // DECAY_TOKENS x the rank rounded up to a multiple of 4
+  const int stride = (rank + 3) & ~3;
   const int t0 = blockIdx.x * DECAY_TOKENS;
   const int count = tokens - t0 < DECAY_TOKENS ? tokens - t0 : DECAY_TOKENS;
-  for (int e = threadIdx.x; e < DECAY_TOKENS * rank; e += DECAY_NT) {
-    const int tt = e / rank, j = e - tt * rank;
-    const float l = tt < count ? proj[(size_t)(t0 + tt) * proj_stride + low_offset + j] : 0.f;
+  for (int e = threadIdx.x; e < DECAY_TOKENS * stride; e += DECAY_NT) {
+    const int tt = e / stride, j = e - tt * stride;
+    const float l = tt < count && j < rank ? proj[(size_t)(t0 + tt) * proj_stride + low_offset + j] : 0.f;
     low[e] = inv_tau > 0.f ? l : tanhf(l);
   }
   __syncthreads();
@@ -55,11 +56,19 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
   float z[DECAY_TOKENS];
 #pragma unroll
   for (int tt = 0; tt < DECAY_TOKENS; ++tt) z[tt] = 0.f;
-#pragma unroll 8
-  for (int j = 0; j < rank; ++j) {  // ascending j: the order depends on the rank alone
-    const float w = w2t[(size_t)j * channels + c];
+#pragma unroll 4
+  for (int j = 0; j < rank; j += 4) {  // ascending j: the order depends on the rank alone
+    float w[4];
 #pragma unroll
-    for (int tt = 0; tt < DECAY_TOKENS; ++tt) z[tt] = fmaf(w, low[tt * rank + j], z[tt]);
+    for (int i = 0; i < 4; ++i) w[i] = j + i < rank ? w2t[(size_t)(j + i) * channels + c] : 0.f;
+#pragma unroll
+    for (int tt = 0; tt < DECAY_TOKENS; ++tt) {
+      const float4 l = *reinterpret_cast<const float4*>(low + tt * stride + j);
+      z[tt] = fmaf(w[0], l.x, z[tt]);
+      z[tt] = fmaf(w[1], l.y, z[tt]);
+      z[tt] = fmaf(w[2], l.z, z[tt]);
+      z[tt] = fmaf(w[3], l.w, z[tt]);
+    }
   }
   const float b = bias[c];
 #pragma unroll
@@ -234,7 +243,7 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
     copies_wait<STAGES - 1>();  // all but the newest STAGES - 1 groups: this chunk has landed
     __syncthreads();
     const float* chunk = stage + (size_t)buf * CHUNK * row;
-    for (int tt = 0; tt < count; ++tt) {
+    auto walk = [&](int tt) {
       const float* tok = chunk + tt * row;
       const float4* q4 = reinterpret_cast<const float4*>(tok);
       const float4* k4 = reinterpret_cast<const float4*>(tok + DK);
@@ -272,6 +281,12 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
       o += __shfl_xor_sync(0xffffffffu, o, 2);
       if (KS == 8) o += __shfl_xor_sync(0xffffffffu, o, 4);
       if (on && part == 0) out[(size_t)(base + tt) * hv + h * vdim + col] = o * qscale;
+    };
+    if (count == CHUNK) {  // a whole chunk: the next tokens' shared-memory reads and shuffles overlap this one's arithmetic
+#pragma unroll
+      for (int tt = 0; tt < CHUNK; ++tt) walk(tt);
+    } else {
+      for (int tt = 0; tt < count; ++tt) walk(tt);
     }
     __syncthreads();  // the stage is free for the chunk after the next
   }
@@ -311,6 +326,60 @@ gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ proj, i
   }
 }
 
+// The same with LANES lanes an item, four neighbouring entries a lane at a time (vdim a multiple of 4, everything 16-byte
+// aligned): a warp takes 32 / LANES heads at once.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(FINISH_WARPS * 32)
+gla_finish_wide_kernel(const float* __restrict__ o, const float* __restrict__ proj, int proj_stride, int gate_offset,
+                       const float* __restrict__ weight, int weight_stride, T* __restrict__ out, long long items, int heads,
+                       int vdim, float eps) {
+  tl::pdl_launch_dependents();
+  tl::pdl_wait();
+  constexpr int KEEP = LANES == 32 ? 2 : 1;  // quads of a lane: vdim up to 4 LANES KEEP
+  const int sub = threadIdx.x % LANES;
+  const long long item = ((long long)blockIdx.x * FINISH_WARPS * 32 + threadIdx.x) / LANES;
+  const bool live = item < items;
+  const long long t = live ? item / heads : 0;
+  const int h = live ? (int)(item % heads) : 0;
+  const int hv = heads * vdim;
+  const float* row = o + (size_t)t * hv + h * vdim;
+  const float* gate = proj + (size_t)t * proj_stride + gate_offset + h * vdim;
+  float4 v[KEEP], g[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < KEEP; ++n) {
+    const int i = (sub + n * LANES) * 4;
+    v[n] = g[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (live && i < vdim) {
+      v[n] = *reinterpret_cast<const float4*>(row + i);
+      g[n] = *reinterpret_cast<const float4*>(gate + i);
+    }
+    ss = fmaf(v[n].x, v[n].x, ss);
+    ss = fmaf(v[n].y, v[n].y, ss);
+    ss = fmaf(v[n].z, v[n].z, ss);
+    ss = fmaf(v[n].w, v[n].w, ss);
+  }
+#pragma unroll
+  for (int m = LANES / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  const float inv = 1.f / sqrtf(ss / (float)vdim + eps);
+#pragma unroll
+  for (int n = 0; n < KEEP; ++n) {
+    const int i = (sub + n * LANES) * 4;
+    if (!live || i >= vdim) continue;
+    float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (weight) w = *reinterpret_cast<const float4*>(weight + h * weight_stride + i);
+    const float r[4] = {v[n].x * inv * w.x * (g[n].x / (1.f + expf(-g[n].x))), v[n].y * inv * w.y * (g[n].y / (1.f + expf(-g[n].y))),
+                        v[n].z * inv * w.z * (g[n].z / (1.f + expf(-g[n].z))), v[n].w * inv * w.w * (g[n].w / (1.f + expf(-g[n].w)))};
+    T* dst = out + (size_t)t * hv + h * vdim + i;
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+    } else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+      *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+    }
+  }
+}
+
 // Split-half rotation of the first ``dims`` entries of ``heads`` consecutive heads of ``dim`` entries in float32
 // rows, in place: entry i (< dims / 2) pairs with i + dims / 2, angle = float(position) * inv_freq[i].
 __global__ void rotate_heads_kernel(float* __restrict__ rows, int stride, const int* __restrict__ positions,
@@ -344,7 +413,7 @@ int tl_gla_decay(const float* proj, int proj_stride, int low_offset, const float
   if (channels <= 0 || rank <= 0 || rank > 1024 || !(tau >= 0.f)) return TL_ERR_UNSUPPORTED;
   dim3 grid((tokens + DECAY_TOKENS - 1) / DECAY_TOKENS, (channels + DECAY_NT - 1) / DECAY_NT);
   if (grid.y > 65535) return TL_ERR_UNSUPPORTED;
-  tl::launch_kernel(gla_decay_kernel, grid, DECAY_NT, (size_t)DECAY_TOKENS * rank * sizeof(float), stream, proj,
+  tl::launch_kernel(gla_decay_kernel, grid, DECAY_NT, (size_t)DECAY_TOKENS * ((rank + 3) & ~3) * sizeof(float), stream, proj,
                     proj_stride, low_offset, w2t, bias, decay, tokens, channels, rank, tau > 0.f ? 1.f / tau : 0.f);
   return TL_LAUNCH_CHECK();
 }
@@ -403,6 +472,24 @@ int tl_gla_finish(const float* o, const float* proj, int proj_stride, int gate_o
                   int out_dtype, int tokens, int heads, int vdim, float eps, cudaStream_t stream) {
   const long long items = (long long)tokens * heads;
   if (items <= 0) return 0;
+  const uintptr_t all = (uintptr_t)o | (uintptr_t)(proj + gate_offset) | (uintptr_t)weight | (uintptr_t)out;
+  if (vdim % 4 == 0 && vdim <= 256 && proj_stride % 4 == 0 && (all & 15) == 0) {
+#define TL_FINISH_WIDE(T, LANES)                                                                                        \
+  tl::launch_kernel(gla_finish_wide_kernel<T, LANES>, (unsigned)((items * LANES + FINISH_WARPS * 32 - 1) / (FINISH_WARPS * 32)), \
+                    FINISH_WARPS * 32, 0, stream, o, proj, proj_stride, gate_offset, weight, weight_stride, (T*)out, items, heads, \
+                    vdim, eps)
+    if (out_dtype == TL_DTYPE_F32) {
+      if (vdim <= 32) TL_FINISH_WIDE(float, 8);
+      else if (vdim <= 64) TL_FINISH_WIDE(float, 16);
+      else TL_FINISH_WIDE(float, 32);
+    } else {
+      if (vdim <= 32) TL_FINISH_WIDE(__nv_bfloat16, 8);
+      else if (vdim <= 64) TL_FINISH_WIDE(__nv_bfloat16, 16);
+      else TL_FINISH_WIDE(__nv_bfloat16, 32);
+    }
+#undef TL_FINISH_WIDE
+    return TL_LAUNCH_CHECK();
+  }
   const unsigned blocks = (unsigned)((items + FINISH_WARPS - 1) / FINISH_WARPS);
   if (out_dtype == TL_DTYPE_F32)
     tl::launch_kernel(gla_finish_kernel<float>, blocks, FINISH_WARPS * 32, 0, stream, o, proj, proj_stride,

@@ -5,8 +5,8 @@
 //   acc += m * norm(v) (+ row)                                         norm: layer norm or RMS norm, weight (and bias)
 //   out = norm'(acc) in the compute type                               (optional) what the next sub-layer reads
 //
-// A row is kept in registers from the first load to the last store: one trip to memory, four block sums.  The order of
-// the additions depends on the width alone.  ``y`` may be left zeroed for the next sub-layer to add into.
+// A row is kept in registers from the first load to the last store: one trip to memory, four block sums.  Without split
+// sums (the 32-bit engine has none) the order of the additions depends on the width alone.  ``y`` may be left zeroed for the next sub-layer to add into.
 //
 //   add_row        acc[t] += row for every token
 //   relu_squared   x = max(x, 0)^2 in place (where the product before it has no such epilogue)
@@ -57,21 +57,27 @@ template <int V> __device__ __forceinline__ void store_v(__nv_bfloat16* p, const
   }
 }
 
-// sum += the ``count`` planes of src at the thread's entries, PER loads in flight.
+// sum += the ``count`` planes of src at the thread's entries, in ascending order, all of eight planes' loads of an entry
+// in flight: a step of few tokens is a chain of dependent trips to memory.
 template <int NT, int PER, int V>
 __device__ __forceinline__ void add_planes(float (&sum)[PER][V], const float* src, int count, size_t plane, int width) {
-  for (int s = 0; s < count; ++s) {
-    float part[PER][V];
+  constexpr int BATCH = 8;
+  for (int s0 = 0; s0 < count; s0 += BATCH) {
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int j = (threadIdx.x + k * NT) * V;
-      if (j < width) load_v<V>(src + s * plane + j, part[k]);
-    }
+      if (j < width) {
+        float part[BATCH][V];
 #pragma unroll
-    for (int k = 0; k < PER; ++k) {
-      if ((threadIdx.x + k * NT) * V < width) {
+        for (int s = 0; s < BATCH; ++s) {
 #pragma unroll
-        for (int e = 0; e < V; ++e) sum[k][e] += part[k][e];
+          for (int e = 0; e < V; ++e) part[s][e] = 0.f;
+          if (s0 + s < count) load_v<V>(src + (s0 + s) * plane + j, part[s]);
+        }
+#pragma unroll
+        for (int s = 0; s < BATCH; ++s)
+#pragma unroll
+          for (int e = 0; e < V; ++e) sum[k][e] += part[s][e];
       }
     }
   }
@@ -103,8 +109,8 @@ __device__ __forceinline__ float2 moments(const float (&v)[PER][V], int width, f
   return make_float2(mean, 1.f / sqrtf(block_sum<NT>(ss, scratch) / (float)width + eps));
 }
 
-// One block a row; a thread holds PER x V entries of it.
-template <typename T, int NT, int PER, int V>
+// One block a row; a thread holds PER x V entries of it.  SUMS: y or the gate comes with split sums.
+template <typename T, int NT, int PER, int V, bool SUMS>
 __global__ void __launch_bounds__(NT)
 residual_norm_kernel(const Args a) {
   tl::pdl_launch_dependents();
@@ -133,8 +139,10 @@ residual_norm_kernel(const Args a) {
       if (a.gate) load_v<V>(a.gate + at + j, g[k]);
     }
   }
-  add_planes<NT, PER, V>(v, a.partials + at, a.splits, a.plane, a.width);
-  if (a.gate) add_planes<NT, PER, V>(g, a.gate + a.plane + at, a.gate_splits - 1, a.plane, a.width);
+  if constexpr (SUMS) {
+    add_planes<NT, PER, V>(v, a.partials + at, a.splits, a.plane, a.width);
+    if (a.gate) add_planes<NT, PER, V>(g, a.gate + a.plane + at, a.gate_splits - 1, a.plane, a.width);
+  }
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
     const int j = (threadIdx.x + k * NT) * V;
@@ -215,18 +223,27 @@ int launch_residual(const Args& a, int rows, cudaStream_t stream) {
                         (uintptr_t)a.gate_bias | (uintptr_t)a.weight | (uintptr_t)a.bias | (uintptr_t)a.row |
                         (uintptr_t)a.out | (uintptr_t)a.weight2 | (uintptr_t)a.bias2;
   const bool wide = a.width % 4 == 0 && (all & 15) == 0;
-#define TL_RESIDUAL(NT, PER, V) tl::launch_kernel(residual_norm_kernel<T, NT, PER, V>, (unsigned)rows, NT, 0, stream, a)
-  if (wide) {
-    if (a.width <= 1024) TL_RESIDUAL(256, 1, 4);
-    else if (a.width <= 2048) TL_RESIDUAL(256, 2, 4);
-    else if (a.width <= 4096) TL_RESIDUAL(512, 2, 4);
-    else if (a.width <= 8192) TL_RESIDUAL(512, 4, 4);
-    else if (a.width <= 16384) TL_RESIDUAL(1024, 4, 4);
+  const bool sums = a.splits > 0 || (a.gate && a.gate_splits > 1);
+#define TL_RESIDUAL(NT, PER, V)                                                                               \
+  {                                                                                                           \
+    if (sums) tl::launch_kernel(residual_norm_kernel<T, NT, PER, V, true>, (unsigned)rows, NT, 0, stream, a); \
+    else tl::launch_kernel(residual_norm_kernel<T, NT, PER, V, false>, (unsigned)rows, NT, 0, stream, a);     \
+  }
+  if (wide && sums && a.width <= 4096 && rows <= 512) {  // few rows: one round of loads a thread
+    if (a.width <= 1024) TL_RESIDUAL(256, 1, 4)
+    else if (a.width <= 2048) TL_RESIDUAL(512, 1, 4)
+    else TL_RESIDUAL(1024, 1, 4)
+  } else if (wide) {
+    if (a.width <= 1024) TL_RESIDUAL(256, 1, 4)
+    else if (a.width <= 2048) TL_RESIDUAL(256, 2, 4)
+    else if (a.width <= 4096) TL_RESIDUAL(512, 2, 4)
+    else if (a.width <= 8192) TL_RESIDUAL(512, 4, 4)
+    else if (a.width <= 16384) TL_RESIDUAL(1024, 4, 4)
     else return TL_ERR_UNSUPPORTED;
   } else {
-    if (a.width <= 1024) TL_RESIDUAL(256, 4, 1);
-    else if (a.width <= 4096) TL_RESIDUAL(512, 8, 1);
-    else if (a.width <= 16384) TL_RESIDUAL(1024, 16, 1);
+    if (a.width <= 1024) TL_RESIDUAL(256, 4, 1)
+    else if (a.width <= 4096) TL_RESIDUAL(512, 8, 1)
+    else if (a.width <= 16384) TL_RESIDUAL(1024, 16, 1)
     else return TL_ERR_UNSUPPORTED;
   }
 #undef TL_RESIDUAL

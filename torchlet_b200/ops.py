@@ -59,6 +59,7 @@ _SIGNATURES = {
                              c_longlong, c_void_p, c_longlong, c_int, c_void_p],
         "tl_gemm_tc_grouped": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                                c_float, c_float, c_void_p],
+        "tl_gemm_tc_stacked": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p, c_void_p],
         "tl_gemm_tc_plan": [c_int, c_int, c_int, c_void_p, c_void_p],
         "tl_gemm_tc_error": [],
         "tl_gemm_tc_wait_selftest": [c_int, c_void_p],
@@ -183,6 +184,12 @@ _SIGNATURES = {
                              c_int, c_int, c_void_p],
         "tl_add_row": [c_void_p, c_void_p, c_int, c_int, c_void_p],
         "tl_relu_squared": [c_void_p, c_int, c_longlong, c_void_p],
+    },
+    "time_mixing": {
+        "tl_time_mixing_step_supported": [c_int, c_int, c_int],
+        "tl_time_mixing_step": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
+        "tl_time_mixing_debug_error": [c_void_p],
     },
     "token_shift": {
         "tl_token_shift": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p,
@@ -766,6 +773,49 @@ def token_shift(x, mu, out, state, token_req, req_indptr, slots, requests: int) 
         x.data_ptr(), dtype_code(x.dtype), mu.data_ptr(), n, out.data_ptr(), out.stride(0), state.data_ptr(), state.shape[0],
         token_req.data_ptr(), req_indptr.data_ptr(), slots.data_ptr(), requests, tokens, width, _stream())
     _check(code, "token_shift")
+
+
+STACKED_ROWS = (16, 32, 64)  # rows a group of ``gemm_tc_stacked`` may have
+
+
+def gemm_tc_stacked(x, w, N: int):
+    """Products of few rows each as one launch: x [groups, rows, K] bfloat16 (rows 16, 32 or 64), w [stack rows, K] with
+    group g's matrix in rows [g N, (g + 1) N) (the last group may have fewer).  Left as float32 partial sums
+    [splits, groups * rows, N] in the shared workspace for a finishing kernel; returns (partials, splits).  Columns past
+    the rows of a short last group are not written."""
+    _need_cuda(x, w)
+    _release_workspace()
+    groups, rows, K = x.shape
+    assert x.dtype == w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and w.shape[1] == K
+    splits = ctypes.c_int(0)
+    fn = _fn("gemm_tc", "tl_gemm_tc_stacked")
+    args = (x.data_ptr(), w.data_ptr(), groups, rows, N, K, w.shape[0])
+    code = fn(*args, None, 0, ctypes.byref(splits), _stream())
+    if code == 0:
+        ws = _workspace(x.device, splits.value * groups * rows * N * 4)
+        code = fn(*args, ws.data_ptr(), ws.numel() * 4, ctypes.byref(splits), _stream())
+    _check(code, "gemm_tc_stacked")
+    return ws, splits.value
+
+
+def time_mixing_step_supported(heads: int, dim: int, rank: int) -> bool:
+    return bool(_fn("time_mixing", "tl_time_mixing_step_supported")(heads, dim, rank))
+
+
+def time_mixing_step(sums, splits: int, group_rows: int, w2t, w0, bonus, weight, slots, state, out, heads: int, dim: int,
+                     eps: float) -> None:
+    """One token a request of a time-mixing recurrence, from the split sums of its products (``gemm_tc_stacked`` over r,
+    k, v, g and the decay's low-rank input) to the normed and gated heads ``out`` (bfloat16); the slots' states move on
+    (csrc/time_mixing.cu)."""
+    _need_cuda(sums, w2t, w0, bonus, weight, slots, state, out)
+    rank, size = w2t.shape
+    assert size == heads * dim and all(t.dtype == torch.float32 and t.is_contiguous() for t in (sums, w2t, w0, bonus, weight, state))
+    assert state.shape[1:] == (heads, dim, dim) and out.is_contiguous() and out.dtype == torch.bfloat16 and out.shape[1] == size
+    assert sums.numel() >= splits * 5 * group_rows * size and slots.dtype == torch.int32
+    code = _fn("time_mixing", "tl_time_mixing_step")(
+        sums.data_ptr(), splits, group_rows, w2t.data_ptr(), w0.data_ptr(), bonus.data_ptr(), weight.data_ptr(), slots.data_ptr(),
+        state.data_ptr(), out.data_ptr(), out.shape[0], heads, dim, rank, state.shape[0], float(eps), _stream())
+    _check(code, "time_mixing_step")
 
 
 # ------------------------------ attention over a window of tokens and pooled blocks of older ones
@@ -1464,7 +1514,7 @@ def debug_errors() -> list:
     found = []
     for library in ("elementwise", "attention_generic", "attention_mma", "decode_fused", "slots", "stream_ops",
                     "delta_rule", "latent_attention", "latent_attention_mma", "gla", "gated_attention", "hyper",
-                    "pooled_attention", "ssm", "token_shift"):
+                    "pooled_attention", "ssm", "time_mixing", "token_shift"):
         if any(name in _functions for name in _SIGNATURES[library]):
             value = ctypes.c_int(0)
             code = _fn(library, f"tl_{library}_debug_error")(ctypes.byref(value))

@@ -149,7 +149,11 @@ class GatedAttentionMixer(Mixer):
 
         sizes = {"q": (self.qk_dim, order), "k": (self.qk_dim, order), "v": (self.v_dim, v_order),
                  "g": (1, None) if self.gate == "head_sigmoid" else (self.v_dim, v_order)}
-        self.in_proj = Linear(torch.cat([heads_of(n, *sizes[n]) for n in names], dim=0), None, device, dtype)
+        rows = [heads_of(n, *sizes[n]) for n in names]
+        odd = -sum(w.shape[0] for w in rows) % 4
+        if odd:  # zero rows behind the last: float32 output rows of whole 16-byte pieces
+            rows.append(rows[-1].new_zeros(odd, rows[-1].shape[1]))
+        self.in_proj = Linear(torch.cat(rows, dim=0), None, device, dtype)
         w_o = tensors[prefix + "o"]
         if v_order is not None and v_order != list(range(self.v_dim)):  # the heads' outputs come in the values' order
             w_o = w_o.reshape(w_o.shape[0], self.num_heads, self.v_dim)[:, :, v_order].reshape(w_o.shape[0], -1)

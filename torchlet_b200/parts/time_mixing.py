@@ -11,7 +11,8 @@ gate = silu(W_g m_g), and a decay per key channel a = exp(-exp(W_w2 tanh(W_w1 m_
 Each head's o is divided by its root mean square; the heads, concatenated, are multiplied by a weight over all of them
 and by the gate, and go through W_o into the stream.  The products r, k, v and g run over the mixes' planes and leave
 float32 planes, which the scan of the gated linear attention reads (csrc/gla.cu); decay, state, recurrence and norm are
-float32 in both engines.
+float32 in both engines.  A step of single tokens in bfloat16 runs all five products as one launch over the stacked
+matrices and everything from their split sums to the gated heads as one kernel (csrc/time_mixing.cu).
 
 Parameters: ``hidden_size``, ``num_heads``, ``head_dim``, ``decay_rank``, ``eps``.  Tensors below the prefix: r, k, v, g
 [H D, hidden]; w1 [rank, hidden]; w2 [H D, rank]; w0, norm [H D]; u [H, D]; mu.r, mu.k, mu.v, mu.g, mu.w [hidden];
@@ -47,6 +48,7 @@ class TimeMixing(Mixer):
         if self.rank > 1024:
             raise ValueError(f"a decay rank of {self.rank} is not supported (up to 1024)")
         self.size = self.num_heads * self.head_dim
+        self.stacked = None  # [4 H D + rank, hidden]: the five input matrices; the products below are views of it
         self.products: list = []
         self.w1_proj: Linear | None = None
         self.o_proj: Linear | None = None
@@ -68,8 +70,12 @@ class TimeMixing(Mixer):
         return out
 
     def load(self, tensors: dict, prefix: str, device, dtype) -> None:
-        self.products = [Linear(tensors[prefix + c], None, device, dtype) for c in PRODUCTS]
-        self.w1_proj = Linear(tensors[prefix + "w1"], None, device, dtype)
+        self.stacked = torch.cat([tensors[prefix + c] for c in PRODUCTS] + [tensors[prefix + "w1"]]).to(
+            device=device, dtype=dtype).contiguous()
+        self.products = [Linear.from_device_weight(self.stacked[i * self.size:(i + 1) * self.size]) for i in range(len(PRODUCTS))]
+        self.w1_proj = Linear.from_device_weight(self.stacked[len(PRODUCTS) * self.size:])
+        self.one_kernel = (dtype == torch.bfloat16 and self.hidden_size % 8 == 0
+                           and ops.time_mixing_step_supported(self.num_heads, self.head_dim, self.rank))
         self.o_proj = Linear(tensors[prefix + "o"], None, device, dtype)
         f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
         self.mu = f32(torch.stack([tensors[f"{prefix}mu.{c}"] for c in MIXES]))
@@ -78,11 +84,23 @@ class TimeMixing(Mixer):
 
     def forward(self, ctx, x, acc, cache) -> None:
         tokens, H, D = x.shape[0], self.num_heads, self.head_dim
-        capacity = max(ctx.token_capacity, tokens)  # scratch sized once for the largest step: its addresses never change
+        # scratch sized once for the largest step: its addresses never change
+        capacity = max(ctx.token_capacity, tokens, ops.STACKED_ROWS[-1])
 
-        def planes_of(name: str, count: int, width: int, dtype):
-            return ctx.buffer(name, (count * capacity, width), dtype)[:count * tokens].view(count, tokens, width)
+        def planes_of(name: str, count: int, width: int, dtype, rows: int = tokens):
+            return ctx.buffer(name, (count * capacity, width), dtype)[:count * rows].view(count, rows, width)
 
+        out = ctx.buffer("time_mixing.out", (tokens, self.size), ctx.dtype)
+        if self.one_kernel and ctx.decode_only and tokens <= ops.STACKED_ROWS[-1]:
+            rows = next(n for n in ops.STACKED_ROWS if tokens <= n)
+            mixes = planes_of("time_mixing.mixes", len(MIXES), self.hidden_size, ctx.dtype, rows)
+            ops.token_shift(x, self.mu, mixes, cache.state["shift"], ctx.token_req, ctx.req_indptr, ctx.slots, ctx.num_requests)
+            sums, splits = ops.gemm_tc_stacked(mixes, self.stacked, self.size)
+            ops.time_mixing_step(sums, splits, rows, self.w2, self.w0, self.bonus, self.norm_weight, ctx.slots,
+                                 cache.state["matrix"], out, H, D, self.eps)
+            if not self.o_proj.accumulate_later(ctx, out, acc):
+                self.o_proj.forward(out, acc, accumulate=True)
+            return
         mixes = planes_of("time_mixing.mixes", len(MIXES), self.hidden_size, ctx.dtype)
         ops.token_shift(x, self.mu, mixes, cache.state["shift"], ctx.token_req, ctx.req_indptr, ctx.slots, ctx.num_requests)
         planes = planes_of("time_mixing.planes", len(PRODUCTS), self.size, torch.float32)
@@ -96,7 +114,6 @@ class TimeMixing(Mixer):
         plane = tokens * self.size
         ops.gla_scan(planes[0], decay, ctx.req_indptr, ctx.slots, cache.state["matrix"], o, ctx.num_requests, H, D, D, 1.0,
                      bonus=self.bonus, k_offset=plane, v_offset=2 * plane)
-        out = ctx.buffer("time_mixing.out", (tokens, self.size), ctx.dtype)
         ops.gla_finish(o, planes[3], 0, self.norm_weight, out, H, D, self.eps)
         if not self.o_proj.accumulate_later(ctx, out, acc):
             self.o_proj.forward(out, acc, accumulate=True)
