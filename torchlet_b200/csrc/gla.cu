@@ -14,7 +14,7 @@
 // whose decay is a = exp(-exp(z)), z = W2 tanh(l) + b.
 //
 // Three kernels:
-//   decay   one block per (8 tokens, 128 channels): a of every key channel;
+//   decay   one block per (8 tokens, 256 channels): a of every key channel;
 //   scan    one block per (request, head, 32 value channels): the columns of S are independent of one
 //           another; four lanes share a column, each keeps a quarter of it in registers, and the block
 //           walks the request's tokens of this step in order; q, k, a, v of a few tokens at a time are
@@ -32,10 +32,10 @@ namespace {
 using namespace tl;
 
 constexpr int DECAY_TOKENS = 8;
-constexpr int DECAY_NT = 128;
+constexpr int DECAY_NT = 256;
 
 // w2t: W2 transposed, [rank, channels]; out: [tokens, channels].
-__global__ void __launch_bounds__(DECAY_NT)
+__global__ void __launch_bounds__(DECAY_NT, 4)
 gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset, const float* __restrict__ w2t,
                  const float* __restrict__ bias, float* __restrict__ out, int tokens, int channels, int rank,
                  float inv_tau) {  // inv_tau > 0: sigmoid(z)^(inv_tau); 0: exp(-exp(z)) of a tanh of the low-rank input
@@ -56,7 +56,7 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
   float z[DECAY_TOKENS];
 #pragma unroll
   for (int tt = 0; tt < DECAY_TOKENS; ++tt) z[tt] = 0.f;
-#pragma unroll 4
+#pragma unroll 2
   for (int j = 0; j < rank; j += 4) {  // ascending j: the order depends on the rank alone
     float w[4];
 #pragma unroll
@@ -105,10 +105,12 @@ template <int N> __device__ __forceinline__ void copies_wait() {
 // the block walks one chunk, the next three are on their way (a chunk's copies take longer than its
 // arithmetic).  A token costs a block 3 DK / 4 shared-memory reads of 16 bytes a warp, which is what bounds
 // a block of many warps; hence few columns a block, and more blocks.
-// Lanes that share a column: four, or eight at key sizes from 128 on (a lane's share of the column, and with it the
-// chain of additions a token, stays at most 32 long, and a block has eight warps to hide the chain's waits behind).
-__host__ __device__ constexpr int lanes_a_column(int dk) { return dk >= 128 ? 8 : 4; }
-constexpr int COLS = 32;
+// Lanes that share a column: four, or eight at key sizes from 64 on (a lane's share of the column, and with it the
+// chain of additions a token, stays at most 32 long, and a block has several warps to hide the chain's waits behind).
+__host__ __device__ constexpr int lanes_a_column(int dk) { return dk >= 64 ? 8 : 4; }
+// Value channels a block: 32, or 16 where a step's blocks then still fit the GPU once (one prompt alone): the walk is a
+// chain of dependent steps, and half the warps on twice the SMs walk it faster.
+constexpr int COLS_WIDE = 32, COLS_NARROW = 16;
 constexpr int STAGES = 4;
 
 // MODE says what ``decay`` holds: DECAY_ROWS a row [heads * dim] per token (one number a key channel), DECAY_HEAD one
@@ -118,7 +120,7 @@ constexpr int STAGES = 4;
 // DECAY_BONUS: rows like DECAY_ROWS, and ``bonus`` [heads * dim] weighs the current token's k v^T in its own output.
 // k stands ``k_offset`` numbers behind q, v ``v_offset``.
 constexpr int DECAY_ROWS = 0, DECAY_HEAD = 1, DECAY_TOKEN = 2, DECAY_BONUS = 3;
-template <int DK, bool VEC, int MODE>
+template <int DK, bool VEC, int MODE, int COLS>
 __global__ void __launch_bounds__(lanes_a_column(DK) * COLS)
 gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __restrict__ decay,
                 const int* __restrict__ req_indptr, const int* __restrict__ slots, float* __restrict__ state,
@@ -154,33 +156,51 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
   // entries past dim (and past vdim) stay zero in both stages
   for (int e = tid; e < STAGES * CHUNK * row; e += NT) stage[e] = 0.f;
   __syncthreads();
+  // which pieces of a chunk this thread copies: the same of every chunk, so the addresses are worked out once
+  constexpr int PIECES = (CHUNK * ((FIXED ? 2 : 3) * DK / 4 + COLS / 4 + 1) + NT - 1) / NT;
+  const float* piece_src[PIECES];
+  int piece_to[PIECES], piece_token[PIECES];  // where in a stage; the token of the chunk (CHUNK: none)
+  bool piece_decay[PIECES];
+  if (VEC) {
+    const int qd = dim >> 2, qv = cols_here >> 2, per_token = (FIXED ? 2 : 3) * qd + qv + (MODE == DECAY_TOKEN ? 1 : 0);
+#pragma unroll
+    for (int n = 0; n < PIECES; ++n) {
+      const int e = tid + n * NT, tt = e / per_token, rest = e - tt * per_token;
+      const int t = first + tt;
+      piece_token[n] = tt < CHUNK ? tt : CHUNK;
+      piece_decay[n] = false;
+      if (rest < 2 * qd) {
+        const int what = rest / qd, q4 = rest - what * qd;
+        piece_src[n] = proj + (size_t)t * proj_stride + what * k_offset + hq * dim + 4 * q4;
+        piece_to[n] = tt * row + what * DK + 4 * q4;
+      } else if (!FIXED && rest < 3 * qd) {
+        const int q4 = rest - 2 * qd;
+        piece_src[n] = decay + (size_t)t * heads * dim + h * dim + 4 * q4;
+        piece_to[n] = tt * row + 2 * DK + 4 * q4;
+        piece_decay[n] = true;
+      } else if (MODE == DECAY_TOKEN && rest == per_token - 1) {
+        piece_src[n] = decay + (size_t)t * heads + h;
+        piece_to[n] = tt * row + VOFF + COLS;
+        piece_decay[n] = true;
+      } else {
+        const int q4 = rest - (FIXED ? 2 : 3) * qd;
+        piece_src[n] = proj + (size_t)t * proj_stride + v_offset + h * vdim + col0 + 4 * q4;
+        piece_to[n] = tt * row + VOFF + 4 * q4;
+      }
+    }
+  }
+  const size_t proj_step = (size_t)CHUNK * proj_stride, decay_step = (size_t)CHUNK * heads * (MODE == DECAY_TOKEN ? 1 : dim);
   auto fetch = [&](int base, int buf) {
     const int count = last - base < CHUNK ? last - base : CHUNK;
     float* dst = stage + (size_t)buf * CHUNK * row;
     if (VEC) {
-      const int qd = dim >> 2, qv = cols_here >> 2, per_token = (FIXED ? 2 : 3) * qd + qv + (MODE == DECAY_TOKEN ? 1 : 0);
-      for (int e = tid; e < count * per_token; e += NT) {
-        const int tt = e / per_token, rest = e - tt * per_token;
-        const int t = base + tt;
-        const float* src;
-        float* to;
-        if (rest < 2 * qd) {  // q, k
-          const int what = rest / qd, q4 = rest - what * qd;
-          src = proj + (size_t)t * proj_stride + what * k_offset + hq * dim + 4 * q4;
-          to = dst + tt * row + what * DK + 4 * q4;
-        } else if (!FIXED && rest < 3 * qd) {
-          const int q4 = rest - 2 * qd;
-          src = decay + (size_t)t * heads * dim + h * dim + 4 * q4;
-          to = dst + tt * row + 2 * DK + 4 * q4;
-        } else if (MODE == DECAY_TOKEN && rest == per_token - 1) {
-          copy4(dst + tt * row + VOFF + COLS, decay + (size_t)t * heads + h);
-          continue;
-        } else {
-          const int q4 = rest - (FIXED ? 2 : 3) * qd;
-          src = proj + (size_t)t * proj_stride + v_offset + h * vdim + col0 + 4 * q4;
-          to = dst + tt * row + VOFF + 4 * q4;
+#pragma unroll
+      for (int n = 0; n < PIECES; ++n) {
+        if (piece_token[n] < count) {
+          if (MODE == DECAY_TOKEN && piece_decay[n]) copy4(dst + piece_to[n], piece_src[n]);
+          else copy16(dst + piece_to[n], piece_src[n]);
         }
-        copy16(to, src);
+        piece_src[n] += (!FIXED || MODE == DECAY_TOKEN) && piece_decay[n] ? decay_step : proj_step;
       }
     } else {
       const int per_token = (FIXED ? 2 : 3) * dim + cols_here + (MODE == DECAY_TOKEN ? 1 : 0);
@@ -282,9 +302,69 @@ gla_scan_kernel(const float* __restrict__ proj, int proj_stride, const float* __
       if (KS == 8) o += __shfl_xor_sync(0xffffffffu, o, 4);
       if (on && part == 0) out[(size_t)(base + tt) * hv + h * vdim + col] = o * qscale;
     };
-    if (count == CHUNK) {  // a whole chunk: the next tokens' shared-memory reads and shuffles overlap this one's arithmetic
+    // A whole chunk: the next token's shared-memory reads are under way while this one's arithmetic runs, and the lanes'
+    // shares of all the chunk's outputs meet together, in CHUNK independent shuffles a round.  (Key sizes whose share of a
+    // token would not fit the registers twice walk token by token.)
+    if (PER <= 16 && count == CHUNK) {
+      constexpr int QD = PER <= 16 ? PER / 4 : 1;
+      float4 Q[2][QD], K[2][QD], A[2][QD];
+      float V[2], F[2];
+      auto load = [&](int tt, int w) {
+        const float* tok = chunk + tt * row;
+        const float4* q4 = reinterpret_cast<const float4*>(tok);
+        const float4* k4 = reinterpret_cast<const float4*>(tok + DK);
+        const float4* a4 = reinterpret_cast<const float4*>(tok + 2 * DK);
+        V[w] = tok[VOFF + (on ? col - col0 : 0)];
+        F[w] = MODE == DECAY_TOKEN ? tok[VOFF + COLS] : head_decay;
 #pragma unroll
-      for (int tt = 0; tt < CHUNK; ++tt) walk(tt);
+        for (int n = 0; n < QD; ++n) {
+          Q[w][n] = q4[n * KS + part];
+          K[w][n] = k4[n * KS + part];
+          if (!FIXED) A[w][n] = a4[n * KS + part];
+        }
+      };
+      float O[CHUNK];
+      load(0, 0);
+#pragma unroll
+      for (int tt = 0; tt < CHUNK; ++tt) {
+        const int w = tt & 1;
+        if (tt + 1 < CHUNK) load(tt + 1, w ^ 1);
+        const float v = V[w];
+        float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+#pragma unroll
+        for (int n = 0; n < QD; ++n) {
+          const float4 k = K[w][n], q = Q[w][n];
+          const float4 a = FIXED ? make_float4(F[w], F[w], F[w], F[w]) : A[w][n];
+          if constexpr (MODE == DECAY_BONUS) {
+            const float kx = k.x * v, ky = k.y * v, kz = k.z * v, kw = k.w * v;
+            o0 = fmaf(q.x, fmaf(U[4 * n], kx, S[4 * n]), o0);
+            o1 = fmaf(q.y, fmaf(U[4 * n + 1], ky, S[4 * n + 1]), o1);
+            o2 = fmaf(q.z, fmaf(U[4 * n + 2], kz, S[4 * n + 2]), o2);
+            o3 = fmaf(q.w, fmaf(U[4 * n + 3], kw, S[4 * n + 3]), o3);
+            S[4 * n] = fmaf(a.x, S[4 * n], kx);
+            S[4 * n + 1] = fmaf(a.y, S[4 * n + 1], ky);
+            S[4 * n + 2] = fmaf(a.z, S[4 * n + 2], kz);
+            S[4 * n + 3] = fmaf(a.w, S[4 * n + 3], kw);
+          } else {
+            S[4 * n] = fmaf(k.x, v, a.x * S[4 * n]);
+            S[4 * n + 1] = fmaf(k.y, v, a.y * S[4 * n + 1]);
+            S[4 * n + 2] = fmaf(k.z, v, a.z * S[4 * n + 2]);
+            S[4 * n + 3] = fmaf(k.w, v, a.w * S[4 * n + 3]);
+            o0 = fmaf(q.x, S[4 * n], o0);
+            o1 = fmaf(q.y, S[4 * n + 1], o1);
+            o2 = fmaf(q.z, S[4 * n + 2], o2);
+            o3 = fmaf(q.w, S[4 * n + 3], o3);
+          }
+        }
+        O[tt] = (o0 + o1) + (o2 + o3);
+      }
+#pragma unroll
+      for (int m = 1; m < KS; m <<= 1)
+#pragma unroll
+        for (int tt = 0; tt < CHUNK; ++tt) O[tt] += __shfl_xor_sync(0xffffffffu, O[tt], m);
+#pragma unroll
+      for (int tt = 0; tt < CHUNK; ++tt)
+        if (on && part == tt % KS) out[(size_t)(base + tt) * hv + h * vdim + col] = O[tt] * qscale;
     } else {
       for (int tt = 0; tt < count; ++tt) walk(tt);
     }
@@ -430,23 +510,32 @@ int tl_gla_scan(const float* proj, int proj_stride, const float* decay, const in
   if (qk_heads <= 0 || heads % qk_heads || decay_mode < 0 || decay_mode > 3) return TL_ERR_UNSUPPORTED;
   if ((decay_mode == DECAY_BONUS) != (bonus != nullptr)) return TL_ERR_UNSUPPORTED;
   const bool fixed_decay = decay_mode == DECAY_HEAD || decay_mode == DECAY_TOKEN;
-  dim3 grid(requests, heads, (vdim + COLS - 1) / COLS);
   const bool vec = dim % 4 == 0 && vdim % 4 == 0 && proj_stride % 4 == 0 && k_offset % 4 == 0 && v_offset % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
                    (fixed_decay || (reinterpret_cast<uintptr_t>(decay) & 15) == 0);
-#define TL_SCAN_ONE(DK, VEC, MODE)                                                                                 \
-  tl::launch_kernel(gla_scan_kernel<DK, VEC, MODE>, grid, lanes_a_column(DK) * COLS, 0, stream, proj, proj_stride, decay, req_indptr, \
-                    slots, state, out, heads, qk_heads, dim, vdim, max_slots, qscale, bonus, k_offset, v_offset)
-#define TL_SCAN(DK)                                                                \
-  {                                                                                \
-    if (vec && decay_mode == DECAY_HEAD) TL_SCAN_ONE(DK, true, DECAY_HEAD);        \
-    else if (vec && decay_mode == DECAY_TOKEN) TL_SCAN_ONE(DK, true, DECAY_TOKEN); \
-    else if (vec && decay_mode == DECAY_BONUS) TL_SCAN_ONE(DK, true, DECAY_BONUS); \
-    else if (vec) TL_SCAN_ONE(DK, true, DECAY_ROWS);                               \
-    else if (decay_mode == DECAY_HEAD) TL_SCAN_ONE(DK, false, DECAY_HEAD);         \
-    else if (decay_mode == DECAY_TOKEN) TL_SCAN_ONE(DK, false, DECAY_TOKEN);       \
-    else if (decay_mode == DECAY_BONUS) TL_SCAN_ONE(DK, false, DECAY_BONUS);       \
-    else TL_SCAN_ONE(DK, false, DECAY_ROWS);                                       \
+  static int sms = 0;
+  if (!sms) {
+    int device = 0;
+    cudaGetDevice(&device);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
+  }
+  const bool narrow = vec && (long long)requests * heads * ((vdim + COLS_NARROW - 1) / COLS_NARROW) <= sms;
+#define TL_SCAN_ONE(DK, VEC, MODE, COLS)                                                                                   \
+  tl::launch_kernel(gla_scan_kernel<DK, VEC, MODE, COLS>, dim3(requests, heads, (vdim + COLS - 1) / COLS),                 \
+                    lanes_a_column(DK) * COLS, 0, stream, proj, proj_stride, decay, req_indptr, slots, state, out, heads,  \
+                    qk_heads, dim, vdim, max_slots, qscale, bonus, k_offset, v_offset)
+#define TL_SCAN_MODE(DK, MODE)                                    \
+  {                                                               \
+    if (narrow) TL_SCAN_ONE(DK, true, MODE, COLS_NARROW);         \
+    else if (vec) TL_SCAN_ONE(DK, true, MODE, COLS_WIDE);         \
+    else TL_SCAN_ONE(DK, false, MODE, COLS_WIDE);                 \
+  }
+#define TL_SCAN(DK)                                                    \
+  {                                                                    \
+    if (decay_mode == DECAY_HEAD) TL_SCAN_MODE(DK, DECAY_HEAD)         \
+    else if (decay_mode == DECAY_TOKEN) TL_SCAN_MODE(DK, DECAY_TOKEN)  \
+    else if (decay_mode == DECAY_BONUS) TL_SCAN_MODE(DK, DECAY_BONUS)  \
+    else TL_SCAN_MODE(DK, DECAY_ROWS)                                  \
   }
   if (dim <= 16) TL_SCAN(16)
   else if (dim <= 32) TL_SCAN(32)
@@ -454,6 +543,7 @@ int tl_gla_scan(const float* proj, int proj_stride, const float* decay, const in
   else if (dim <= 128) TL_SCAN(128)
   else TL_SCAN(256)
 #undef TL_SCAN
+#undef TL_SCAN_MODE
 #undef TL_SCAN_ONE
   return TL_LAUNCH_CHECK();
 }
