@@ -14,7 +14,7 @@
 // whose decay is a = exp(-exp(z)), z = W2 tanh(l) + b.
 //
 // Three kernels:
-//   decay   one block per (8 tokens, 256 channels): a of every key channel;
+//   decay   one block per (8 tokens, 128 or 512 channels): a of every key channel;
 //   scan    one block per (request, head, 32 value channels): the columns of S are independent of one
 //           another; four lanes share a column, each keeps a quarter of it in registers, and the block
 //           walks the request's tokens of this step in order; q, k, a, v of a few tokens at a time are
@@ -32,13 +32,16 @@ namespace {
 using namespace tl;
 
 constexpr int DECAY_TOKENS = 8;
-constexpr int DECAY_NT = 256;
+constexpr int DECAY_NT = 128;
 
-// w2t: W2 transposed, [rank, channels]; out: [tokens, channels].
-__global__ void __launch_bounds__(DECAY_NT, 4)
+// w2t: W2 transposed, [rank, channels]; out: [tokens, channels].  TANH: exp(-exp(z)) of a tanh of the low-rank input, else
+// sigmoid(z)^(inv_tau).  A thread takes CH neighbouring channels: four where the grid is large anyway (a shared-memory read
+// of the low-rank input then serves four channels, and those reads are what a long prompt's time goes into), one otherwise.
+template <bool TANH, int CH>
+__global__ void __launch_bounds__(DECAY_NT)
 gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset, const float* __restrict__ w2t,
                  const float* __restrict__ bias, float* __restrict__ out, int tokens, int channels, int rank,
-                 float inv_tau) {  // inv_tau > 0: sigmoid(z)^(inv_tau); 0: exp(-exp(z)) of a tanh of the low-rank input
+                 float inv_tau) {
   tl::pdl_launch_dependents();
   tl::pdl_wait();
   extern __shared__ __align__(16) float low[];  // DECAY_TOKENS x the rank rounded up to a multiple of 4
@@ -48,40 +51,62 @@ gla_decay_kernel(const float* __restrict__ proj, int proj_stride, int low_offset
   for (int e = threadIdx.x; e < DECAY_TOKENS * stride; e += DECAY_NT) {
     const int tt = e / stride, j = e - tt * stride;
     const float l = tt < count && j < rank ? proj[(size_t)(t0 + tt) * proj_stride + low_offset + j] : 0.f;
-    low[e] = inv_tau > 0.f ? l : tanhf(l);
+    low[e] = TANH ? tanhf(l) : l;
   }
   __syncthreads();
-  const int c = blockIdx.y * DECAY_NT + threadIdx.x;
+  const int c = (blockIdx.y * DECAY_NT + threadIdx.x) * CH;
   if (c >= channels) return;
-  float z[DECAY_TOKENS];
+  float z[DECAY_TOKENS][CH];
 #pragma unroll
-  for (int tt = 0; tt < DECAY_TOKENS; ++tt) z[tt] = 0.f;
-#pragma unroll 2
+  for (int tt = 0; tt < DECAY_TOKENS; ++tt)
+#pragma unroll
+    for (int k = 0; k < CH; ++k) z[tt][k] = 0.f;
+#pragma unroll(CH == 1 ? 4 : 1)
   for (int j = 0; j < rank; j += 4) {  // ascending j: the order depends on the rank alone
-    float w[4];
+    float w[4][CH];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) w[i] = j + i < rank ? w2t[(size_t)(j + i) * channels + c] : 0.f;
+    for (int i = 0; i < 4; ++i) {
+      const float* src = w2t + (size_t)(j + i) * channels + c;
+      if constexpr (CH == 4) {
+        const float4 v = j + i < rank ? *reinterpret_cast<const float4*>(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+        w[i][0] = v.x; w[i][1] = v.y; w[i][2] = v.z; w[i][3] = v.w;
+      } else {
+        w[i][0] = j + i < rank ? *src : 0.f;
+      }
+    }
 #pragma unroll
     for (int tt = 0; tt < DECAY_TOKENS; ++tt) {
       const float4 l = *reinterpret_cast<const float4*>(low + tt * stride + j);
-      z[tt] = fmaf(w[0], l.x, z[tt]);
-      z[tt] = fmaf(w[1], l.y, z[tt]);
-      z[tt] = fmaf(w[2], l.z, z[tt]);
-      z[tt] = fmaf(w[3], l.w, z[tt]);
+#pragma unroll
+      for (int k = 0; k < CH; ++k) {
+        z[tt][k] = fmaf(w[0][k], l.x, z[tt][k]);
+        z[tt][k] = fmaf(w[1][k], l.y, z[tt][k]);
+        z[tt][k] = fmaf(w[2][k], l.z, z[tt][k]);
+        z[tt][k] = fmaf(w[3][k], l.w, z[tt][k]);
+      }
     }
   }
-  const float b = bias[c];
+  float b[CH];
+#pragma unroll
+  for (int k = 0; k < CH; ++k) b[k] = bias[c + k];
 #pragma unroll
   for (int tt = 0; tt < DECAY_TOKENS; ++tt) {
     if (tt >= count) break;
-    const float x = z[tt] + b;
-    if (inv_tau == 0.f) {
-      out[(size_t)(t0 + tt) * channels + c] = expf(-expf(x));
-      continue;
+    float a[CH];
+#pragma unroll
+    for (int k = 0; k < CH; ++k) {
+      const float x = z[tt][k] + b[k];
+      if constexpr (TANH) {
+        a[k] = expf(-expf(x));
+      } else {
+        // log(sigmoid(x)) = min(x, 0) - log1p(exp(-|x|))
+        const float logsig = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
+        a[k] = expf(logsig * inv_tau);
+      }
     }
-    // log(sigmoid(x)) = min(x, 0) - log1p(exp(-|x|))
-    const float logsig = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
-    out[(size_t)(t0 + tt) * channels + c] = expf(logsig * inv_tau);
+    float* dst = out + (size_t)(t0 + tt) * channels + c;
+    if constexpr (CH == 4) *reinterpret_cast<float4*>(dst) = make_float4(a[0], a[1], a[2], a[3]);
+    else *dst = a[0];
   }
 }
 
@@ -491,10 +516,20 @@ int tl_gla_decay(const float* proj, int proj_stride, int low_offset, const float
                  int tokens, int channels, int rank, float tau, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (channels <= 0 || rank <= 0 || rank > 1024 || !(tau >= 0.f)) return TL_ERR_UNSUPPORTED;
-  dim3 grid((tokens + DECAY_TOKENS - 1) / DECAY_TOKENS, (channels + DECAY_NT - 1) / DECAY_NT);
+  const int chunks = (tokens + DECAY_TOKENS - 1) / DECAY_TOKENS;
+  const bool four = chunks >= 64 && channels % 4 == 0 && (((uintptr_t)w2t | (uintptr_t)decay) & 15) == 0;
+  const int per_block = DECAY_NT * (four ? 4 : 1);
+  const dim3 grid(chunks, (channels + per_block - 1) / per_block);
   if (grid.y > 65535) return TL_ERR_UNSUPPORTED;
-  tl::launch_kernel(gla_decay_kernel, grid, DECAY_NT, (size_t)DECAY_TOKENS * ((rank + 3) & ~3) * sizeof(float), stream, proj,
-                    proj_stride, low_offset, w2t, bias, decay, tokens, channels, rank, tau > 0.f ? 1.f / tau : 0.f);
+  const size_t smem = (size_t)DECAY_TOKENS * ((rank + 3) & ~3) * sizeof(float);
+#define TL_DECAY(TANH, CH)                                                                                             \
+  tl::launch_kernel(gla_decay_kernel<TANH, CH>, grid, DECAY_NT, smem, stream, proj, proj_stride, low_offset, w2t, bias, decay, \
+                    tokens, channels, rank, tau > 0.f ? 1.f / tau : 0.f)
+  if (tau > 0.f && four) TL_DECAY(false, 4);
+  else if (tau > 0.f) TL_DECAY(false, 1);
+  else if (four) TL_DECAY(true, 4);
+  else TL_DECAY(true, 1);
+#undef TL_DECAY
   return TL_LAUNCH_CHECK();
 }
 
