@@ -9,7 +9,8 @@ Added here: GROUPS of layer executions with different needs.  A group is a set o
 executions whose mixers keep the same kind of history (same KV heads, head size and
 window); it has its own pool of pages and its own table per request.  A group with a
 window gives a page back as soon as every position in it has left the window of the
-request's next token; the table entry then points at page 0 and is never read.
+request's next token, unless the group keeps the sequence's first tokens and the page holds one of
+them; the table entry then points at page 0 and is never read.
 
 This module is host-only bookkeeping (no device memory) so that it can be tested
 without a GPU; ``torchlet_b200.cache.storage`` owns the device tensors.
@@ -38,6 +39,7 @@ class GroupSpec:
     entries: tuple  # schedule entries that own a cache layer in this group
     num_pages: int  # pool size, page 0 included
     planes: int = 2  # rows a token keeps per KV head: key and value, or one latent row
+    keep_first: int = 0  # a windowed group never gives back the pages of a sequence's first that many tokens
 
 
 class PagePool:
@@ -79,7 +81,7 @@ class _RequestPages:
     slot: int
     num_tokens: int = 0  # tokens whose keys and values are in pages (steps done so far)
     tables: list = field(default_factory=list)  # per group: logical page -> physical page
-    first_live: list = field(default_factory=list)  # per group: first logical page still held
+    first_live: list = field(default_factory=list)  # per group: first logical page still held (kept first pages aside)
     capacity: int = 0  # tokens that fit the pages reserved so far, at most the length limit
 
 
@@ -120,7 +122,9 @@ class CacheManager:
             raise CacheError("no free slot")
         slot = self._free_slots.pop()
         self._requests[request_id] = _RequestPages(
-            slot=slot, tables=[[] for _ in self.groups], first_live=[0 for _ in self.groups]
+            slot=slot, tables=[[] for _ in self.groups],
+            # the pages of kept first tokens lie before the first one that may ever be given back
+            first_live=[-(-g.keep_first // self.page_size) for g in self.groups],
         )
         return slot
 

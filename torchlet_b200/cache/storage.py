@@ -32,7 +32,7 @@ class LayerCache:
 
 
 def plan_groups(needs: list, num_pages: int) -> tuple[list[GroupSpec], dict]:
-    """Group the executions that own paged history by (kv_heads, head_dim, window, planes).
+    """Group the executions that own paged history by (kv_heads, head_dim, window, planes, kept first tokens).
     Returns the groups and a map entry -> (group index, layer index inside the group)."""
     keys, members = [], {}
     for need in needs:
@@ -45,7 +45,7 @@ def plan_groups(needs: list, num_pages: int) -> tuple[list[GroupSpec], dict]:
         members[key].append(need.entry)
     groups, where = [], {}
     for g, key in enumerate(keys):
-        groups.append(GroupSpec(key[0], key[1], key[2], tuple(members[key]), num_pages, planes=key[3]))
+        groups.append(GroupSpec(key[0], key[1], key[2], tuple(members[key]), num_pages, planes=key[3], keep_first=key[4]))
         for i, entry in enumerate(members[key]):
             where[entry] = (g, i)
     return groups, where
@@ -53,7 +53,7 @@ def plan_groups(needs: list, num_pages: int) -> tuple[list[GroupSpec], dict]:
 
 class CacheStorage:
     def __init__(self, needs: list, page_size: int, max_slots: int, num_pages: int, max_seq_len: int,
-                 device, dtype: torch.dtype):
+                 device, dtype: torch.dtype, model_state: dict | None = None):
         self.needs = needs
         self.page_size = page_size
         self.groups, self.where = plan_groups(needs, num_pages)
@@ -79,6 +79,7 @@ class CacheStorage:
             return torch.zeros((max_slots, *spec.slot_shape(max_seq_len)), device=device, dtype=getattr(torch, spec.dtype))
 
         self.states, self.block_states = {}, {}
+        self.model_states = make(dict(model_state or {}))  # name -> [max_slots, *shape]: what the model itself keeps a request
         for need in needs:
             if need.state is not None:
                 self.states[need.entry] = make(need.state)
@@ -86,7 +87,7 @@ class CacheStorage:
                 self.block_states[need.entry] = make(need.block_state)
 
     def state_tensors(self) -> list:
-        """Every state tensor (of mixers and of block arrangements), flat."""
+        """Every state tensor (of mixers, of block arrangements and of the model itself), flat."""
         out = []
 
         def walk(held) -> None:
@@ -96,7 +97,7 @@ class CacheStorage:
             elif held is not None:
                 out.append(held)
 
-        for held in (*self.states.values(), *self.block_states.values()):
+        for held in (*self.states.values(), *self.block_states.values(), self.model_states):
             walk(held)
         return out
 

@@ -7,13 +7,14 @@ from .registry import (
     load_config,
     register_architecture,
 )
-from .spec import LayerSpec, ModelSpec, NormSlot, PartSpec, ScheduleEntry
+from .spec import LayerSpec, ModelSpec, NormSlot, PartSpec, ScheduleEntry, TokenPairs
 from .qwen2 import Qwen2Config
 from .dodonex import DodonexConfig
 from .numuzen import NumuzenConfig
 from .fusolix import FusolixConfig
 from .kilatar import KilatarConfig
 from .tekarax import TekaraxConfig
+from .lidizen import LidizenConfig
 
 __all__ = [
     "DodonexConfig",
@@ -21,6 +22,7 @@ __all__ = [
     "FusolixConfig",
     "KilatarConfig",
     "LayerSpec",
+    "LidizenConfig",
     "ModelSpec",
     "NumuzenConfig",
     "NormSlot",
@@ -28,6 +30,7 @@ __all__ = [
     "Qwen2Config",
     "ScheduleEntry",
     "TekaraxConfig",
+    "TokenPairs",
     "architecture_name",
     "ceil_div",
     "config_class_for",

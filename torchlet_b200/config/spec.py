@@ -88,6 +88,19 @@ class ScheduleEntry:
 
 
 @dataclass(frozen=True)
+class TokenPairs:
+    """A second embedding table whose row is chosen by a token AND the one before it in its sequence: row
+    (previous * ``mul_prev`` + token * ``mul_cur``) mod ``buckets`` of ``table_name`` [buckets + 1, hidden]; the last row
+    is that of a sequence's first token.  The row is added to the token's embedding (before an embedding norm); every
+    request's last token is therefore state."""
+
+    table_name: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     architecture: str
     vocab_size: int
@@ -111,6 +124,7 @@ class ModelSpec:
     # a tensor [stream_rows, hidden] whose rows schedule entries add to the stream (``ScheduleEntry.add_row``)
     stream_rows_name: Optional[str] = None
     stream_rows: int = 0
+    token_pairs: Optional[TokenPairs] = None  # a row for every pair of neighbouring tokens, added to the embedding
 
     def validate(self) -> None:
         if not self.layers:

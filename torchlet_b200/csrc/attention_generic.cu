@@ -10,6 +10,11 @@
 // softmax's denominator (a key of score 0 that has no value), or with ``sink_values`` exp(sink_values[head]); ``gate`` (float32 rows) multiplies the
 // output element by element with sigmoid(gate).
 //
+// ``keep`` > 0: the first ``keep`` positions of the sequence are visible beside the window (their tiles come first).
+// ``chunks`` = nkv: a query row spans the keys of ALL KV heads, [nh][nkv][d], and a head's score is the sum over them
+// (scores mixed across the heads, folded into the queries; see csrc/qkv_prepare.cu); 1: the head's own KV head alone.
+// ``v_cols``: how many entries of a value row are written for a head (the cache rows may be padded).
+//
 // This is the true 32-bit kernel and the any-size bfloat16 kernel (head_dim up to 256: keys are
 // read eight entries at a time where head_dim and the query stride are multiples of 8, one at a
 // time otherwise; any head counts, any page size).
@@ -36,11 +41,12 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
                          const int* __restrict__ token_req, const int* __restrict__ positions,
                          T* __restrict__ out, int out_stride, int tokens, int nh, int nkv, int d,
                          int page_size, int window, float scale, int num_pages, float softcap, int sink,
-                         const float* __restrict__ sink_values, const float* __restrict__ gate, int gate_stride, int wide) {
+                         const float* __restrict__ sink_values, const float* __restrict__ gate, int gate_stride, int wide,
+                         int keep, int chunks, int v_cols) {
   tl::pdl_wait();               // everything before us in the stream is complete and visible
   tl::pdl_launch_dependents();  // the next kernel may start its own prologue
 
-  __shared__ float qs[WARPS][MAX_D];
+  extern __shared__ __align__(16) float all_queries[];  // [WARPS][chunks d]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long item = (long long)blockIdx.x * WARPS + warp;
   if (item >= (long long)tokens * nh) return;
@@ -50,12 +56,15 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
   const int lo = first_key(pos, window);
   const int* table = block_table + (size_t)token_req[t] * table_width;
 
-  const T* qrow = q + (size_t)t * q_stride + (size_t)h * d;
-  for (int i = lane; i < d; i += 32) qs[warp][i] = to_float(qrow[i]);
+  const int q_len = chunks * d;
+  float* qs = all_queries + warp * q_len;
+  const T* qrow = q + (size_t)t * q_stride + (size_t)h * q_len;
+  for (int i = lane; i < q_len; i += 32) qs[i] = to_float(qrow[i]);
   __syncwarp();
 
   const size_t page_elems = (size_t)2 * nkv * page_size * d;
-  const size_t k_off = (size_t)kvh * page_size * d;
+  const size_t k_off = chunks > 1 ? 0 : (size_t)kvh * page_size * d;
+  const size_t head_step = (size_t)page_size * d;  // from a key to the next KV head's
   const size_t v_off = ((size_t)nkv + kvh) * page_size * d;
 
   // the sink is a key of a given score (0, or the head's own number) and no value that every query sees: the running
@@ -65,9 +74,13 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
 #pragma unroll
   for (int c = 0; c < MAX_D / 32; ++c) acc[c] = 0.f;
 
-  for (int start = lo & ~31; start <= pos; start += 32) {
+  // tiles of kept first positions that lie wholly before the window's first tile, then the window's
+  const int window_start = lo & ~31;
+  const int kept_end = keep < window_start ? (keep + 31) & ~31 : window_start;
+  for (int start = kept_end > 0 ? 0 : window_start; start <= pos;
+       start = start + 32 == kept_end ? window_start : start + 32) {
     const int key = start + lane;
-    const bool valid = key >= lo && key <= pos;
+    const bool valid = (key >= lo || key < keep) && key <= pos;
     float s = -INFINITY;
     size_t row_off = 0;
     if (valid) {
@@ -77,15 +90,18 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
       row_off = (size_t)page * page_elems + (size_t)(key % page_size) * d;
       const T* krow = pages + row_off + k_off;
       float dot = 0.f;
-      if (wide) {
-        for (int i = 0; i < d; i += 8) {
-          float kv[8];
-          load8(krow + i, kv);
+      for (int c = 0; c < chunks; ++c, krow += head_step) {
+        const float* qc = qs + c * d;
+        if (wide) {
+          for (int i = 0; i < d; i += 8) {
+            float kv[8];
+            load8(krow + i, kv);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) dot = fmaf(qs[warp][i + j], kv[j], dot);
+            for (int j = 0; j < 8; ++j) dot = fmaf(qc[i + j], kv[j], dot);
+          }
+        } else {  // the same order of additions, one entry at a time
+          for (int i = 0; i < d; ++i) dot = fmaf(qc[i], to_float(krow[i]), dot);
         }
-      } else {  // the same order of additions, one entry at a time
-        for (int i = 0; i < d; ++i) dot = fmaf(qs[warp][i], to_float(krow[i]), dot);
       }
       s = dot * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
@@ -97,9 +113,10 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
     m = new_m;
 #pragma unroll
     for (int c = 0; c < MAX_D / 32; ++c) acc[c] *= corr;
-    const int first = lo > start ? lo - start : 0;
+    const int first = start >= keep && lo > start ? lo - start : 0;  // (a lane without a key has weight 0 and is skipped)
     const int last = pos - start < 31 ? pos - start : 31;
     for (int j = first; j <= last; ++j) {
+      if (keep && !__shfl_sync(0xffffffffu, (int)valid, j)) continue;
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const size_t off = __shfl_sync(0xffffffffu, (unsigned long long)row_off, j);
       const T* vrow = pages + off + v_off;
@@ -110,12 +127,12 @@ attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* __restr
       }
     }
   }
-  T* orow = out + (size_t)t * out_stride + (size_t)h * d;
+  T* orow = out + (size_t)t * out_stride + (size_t)h * v_cols;
   const float inv = 1.f / l;
 #pragma unroll
   for (int c = 0; c < MAX_D / 32; ++c) {
     const int i = lane + 32 * c;
-    if (i < d) {
+    if (i < v_cols) {
       float v = acc[c] * inv;
       if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)t * gate_stride + (size_t)h * d + i]));
       orow[i] = from_float<T>(v);
@@ -132,22 +149,31 @@ extern "C" int tl_attention_generic(const void* q, int q_stride, const void* pag
                                     const int* positions, void* out, int out_stride, int tokens,
                                     int nh, int nkv, int d, int page_size, int window, float scale,
                                     int num_pages, float softcap, int sink, const float* sink_values,
-                                    const float* gate, int gate_stride,
+                                    const float* gate, int gate_stride, int keep, int chunks, int v_cols,
                                     cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (d <= 0 || d > MAX_D || nkv <= 0 || nh % nkv || page_size <= 0) return TL_ERR_UNSUPPORTED;
+  if (keep < 0 || (chunks != 1 && chunks != nkv) || v_cols <= 0 || v_cols > d) return TL_ERR_UNSUPPORTED;
+  const size_t smem = (size_t)WARPS * chunks * d * sizeof(float);
+  if (smem > 200 * 1024) return TL_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) {
+    const cudaError_t err = dtype == TL_DTYPE_F32
+        ? cudaFuncSetAttribute(attention_generic_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
+        : cudaFuncSetAttribute(attention_generic_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err != cudaSuccess) return (int)err;
+  }
   const int wide = d % 8 == 0 && q_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(pages) & 31) == 0;
   const long long items = (long long)tokens * nh;
   const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
   if (dtype == TL_DTYPE_F32)
-    tl::launch_kernel(attention_generic_kernel<float>, blocks, WARPS * 32, 0, stream, 
+    tl::launch_kernel(attention_generic_kernel<float>, blocks, WARPS * 32, smem, stream,
         (const float*)q, q_stride, (const float*)pages, block_table, table_width, token_req,
         positions, (float*)out, out_stride, tokens, nh, nkv, d, page_size, window, scale, num_pages, softcap, sink,
-        sink_values, gate, gate_stride, wide);
+        sink_values, gate, gate_stride, wide, keep, chunks, v_cols);
   else
-    tl::launch_kernel(attention_generic_kernel<__nv_bfloat16>, blocks, WARPS * 32, 0, stream, 
+    tl::launch_kernel(attention_generic_kernel<__nv_bfloat16>, blocks, WARPS * 32, smem, stream,
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)pages, block_table, table_width,
         token_req, positions, (__nv_bfloat16*)out, out_stride, tokens, nh, nkv, d, page_size, window,
-        scale, num_pages, softcap, sink, sink_values, gate, gate_stride, wide);
+        scale, num_pages, softcap, sink, sink_values, gate, gate_stride, wide, keep, chunks, v_cols);
   return TL_LAUNCH_CHECK();
 }

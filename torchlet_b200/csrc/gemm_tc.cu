@@ -1286,7 +1286,7 @@ int tl_gemm_tc_grouped(const void* x, const void* w, void* out, long long ldo, i
                        int groups, const int* plan, int tile_rows, float glu_limit, float glu_alpha,
                        cudaStream_t stream) {
   if (rows <= 0 || N <= 0 || groups <= 0) return 0;
-  if (K <= 0 || K % 8 || !plan || epilogue < 0 || epilogue > 3 || (tile_rows != BLOCK_P && tile_rows != 16) ||
+  if (K <= 0 || K % 8 || !plan || epilogue < 0 || epilogue > EPI_RELU2_BF16 || (tile_rows != BLOCK_P && tile_rows != 16) ||
       rows % tile_rows)
     return TL_ERR_UNSUPPORTED;
   if (tile_rows == 16) {

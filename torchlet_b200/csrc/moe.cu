@@ -2,9 +2,9 @@
 // gated feed-forwards.  Everything is planned on the device, so a step needs no answer from the GPU
 // and a step of single tokens can be captured in a CUDA graph.
 //
-//   route     one warp per token: router logits z = W_r x in float32 (ascending k), scores
+//   route     one warp per token: router logits z = W_r x (+ bias) in float32 (ascending k), scores
 //             sigmoid(z) or softmax(z), the ``top`` largest (the lower index wins a tie), optionally
-//             renormalized to sum 1;
+//             renormalized to sum 1; or the ``top`` largest logits, weighted by the softmax over those alone;
 //   plan      one block: rows per expert, each expert's rows rounded up to whole row tiles of
 //             ``tile`` rows so that a tile of the grouped products belongs to ONE expert; the
 //             position of every (token, choice) in that expert-sorted order; the expert of every tile;
@@ -12,7 +12,8 @@
 //             multiplies the expert's INPUT);
 //   products  out[row] = W_e(row) . in[row] over the sorted rows, CUDA cores, ascending k: with the
 //             gated activation g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit),
-//             over [gate; up] stacked weights, or plain (the down projection, float32 output);
+//             over [gate; up] stacked weights, with the square of relu (an ungated expert's first product),
+//             or plain (the down projection, float32 output);
 //   combine   side[token] += sum over the token's choices, in the order of the choices, of the down
 //             rows (times the weight where it multiplies the OUTPUT).
 //
@@ -52,11 +53,12 @@ __device__ __forceinline__ float router_logit(const Row* __restrict__ row, const
 // ``pick`` (shared memory, ``experts`` floats; may be ``score`` itself): the numbers the choice goes by.  With a
 // ``correction`` (one number an expert) they are score + correction, while the weights stay the scores.  The weights
 // are multiplied by ``scale`` at the end.
+// ``score_mode``: 0 sigmoid, 1 softmax over all, 2 the logits themselves, whose chosen ones the weights are the softmax over.
 __device__ __forceinline__ void choose_experts(float* score, float* pick, const float* __restrict__ correction,
-                                               int experts, int top, int softmax_scores, int renormalize,
+                                               int experts, int top, int score_mode, int renormalize,
                                                int lane, int* __restrict__ choice, float* __restrict__ weight,
                                                int groups, int keep, float renorm_eps, float scale) {
-  if (softmax_scores) {
+  if (score_mode == 1) {
     float m = -INFINITY;
     for (int e = lane; e < experts; e += 32) m = fmaxf(m, score[e]);
     m = warp_max(m);
@@ -64,7 +66,7 @@ __device__ __forceinline__ void choose_experts(float* score, float* pick, const 
     for (int e = lane; e < experts; e += 32) l += expf(score[e] - m);
     l = warp_sum(l);
     for (int e = lane; e < experts; e += 32) score[e] = expf(score[e] - m) / l;
-  } else {
+  } else if (score_mode == 0) {
     for (int e = lane; e < experts; e += 32) score[e] = 1.f / (1.f + expf(-score[e]));
   }
   __syncwarp();
@@ -122,6 +124,16 @@ __device__ __forceinline__ void choose_experts(float* score, float* pick, const 
     }
     __syncwarp();
   }
+  if (score_mode == 2) {  // softmax over the chosen logits
+    float m = -INFINITY;
+    for (int j = lane; j < top; j += 32) m = fmaxf(m, weight[j]);
+    m = warp_max(m);
+    float l = 0.f;
+    for (int j = lane; j < top; j += 32) l += expf(weight[j] - m);
+    l = warp_sum(l);
+    for (int j = lane; j < top; j += 32) weight[j] = expf(weight[j] - m) / l * scale;
+    return;
+  }
   if (renormalize || scale != 1.f)
     for (int j = lane; j < top; j += 32) weight[j] = (renormalize ? weight[j] / (total + renorm_eps) : weight[j]) * scale;
 }
@@ -130,8 +142,9 @@ __device__ __forceinline__ void choose_experts(float* score, float* pick, const 
 // experts w, w + ROUTE_WARPS, ...; the first warp then chooses.
 template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ router, int* __restrict__ choice,
-                 float* __restrict__ weight, int tokens, int hidden, int experts, int top, int softmax_scores,
+moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ router, const float* __restrict__ router_bias,
+                 int* __restrict__ choice,
+                 float* __restrict__ weight, int tokens, int hidden, int experts, int top, int score_mode,
                  int renormalize, int groups, int keep, float renorm_eps, const float* __restrict__ correction,
                  float scale, const float* __restrict__ gate_w, float* __restrict__ gate_out) {
   tl::pdl_launch_dependents();
@@ -146,7 +159,7 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ rou
   __syncthreads();
   for (int e = warp; e < experts; e += ROUTE_WARPS) {
     const float part = router_logit(xrow, router + (size_t)e * hidden, hidden, lane);
-    if (lane == 0) all_scores[e] = part;
+    if (lane == 0) all_scores[e] = router_bias ? part + router_bias[e] : part;
   }
   // a gate of one number a token beside the router (an always-on expert's): sigmoid(gate_w . x), by the last warp
   if (gate_w && warp == ROUTE_WARPS - 1) {
@@ -155,7 +168,7 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ rou
   }
   __syncthreads();
   if (warp != 0) return;
-  choose_experts(all_scores, correction ? picks : all_scores, correction, experts, top, softmax_scores, renormalize, lane,
+  choose_experts(all_scores, correction ? picks : all_scores, correction, experts, top, score_mode, renormalize, lane,
                  choice + (size_t)t * top, weight + (size_t)t * top, groups, keep, renorm_eps, scale);
 }
 
@@ -211,7 +224,7 @@ constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 
 // out[row, n] over the rows of tile blockIdx.y, whose expert the plan names.  GLU: w holds, per
 // expert, [gate (N rows); up (N rows)] and out = act(gate . x, up . x); else out = w_e . x.
-template <typename T, typename OutT, bool GLU>
+template <typename T, typename OutT, bool GLU, bool RELU2 = false>
 __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, OutT* __restrict__ out,
                      const int* __restrict__ plan, int N, int K, float limit, float alpha) {
@@ -282,6 +295,10 @@ moe_gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, OutT* __r
       const int n = n0 + tx * TN + j;
       if (n >= N) continue;
       float v = acc[i][j];
+      if constexpr (RELU2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
       if constexpr (GLU) {
         if (limit > 0.f) {
           const float g = fminf(v, limit);
@@ -355,24 +372,26 @@ int tl_moe_tile_rows() { return BM; }
 // choice int32 [tokens, top], weight float32 [tokens, top]; router float32 [experts, hidden].
 // correction (optional, float32 [experts]): added to the scores for the choice only.  scale: multiplies the weights.
 // gate_w (optional, float32 [hidden]) with gate_out (float32 [tokens]): gate_out[t] = sigmoid(gate_w . x[t]).
-int tl_moe_route(const void* x, int ldx, int dtype, const float* router, int* choice, float* weight, int tokens,
-                 int hidden, int experts, int top, int softmax_scores, int renormalize, int groups, int keep,
+// router_bias (optional, float32 [experts]) is added to the logits; score_mode: see choose_experts.
+int tl_moe_route(const void* x, int ldx, int dtype, const float* router, const float* router_bias, int* choice, float* weight,
+                 int tokens, int hidden, int experts, int top, int score_mode, int renormalize, int groups, int keep,
                  float renorm_eps, const float* correction, float scale, const float* gate_w, float* gate_out,
                  cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > experts) return TL_ERR_UNSUPPORTED;
+  if (experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > experts || score_mode < 0 || score_mode > 2)
+    return TL_ERR_UNSUPPORTED;
   if (groups < 1 || keep < 1 || keep > groups || experts % groups || top > keep * (experts / groups) || groups > 2048)
     return TL_ERR_UNSUPPORTED;
   const unsigned blocks = tokens;
   const size_t smem = (size_t)hidden * sizeof(float);
   if (smem > 48 * 1024) return TL_ERR_UNSUPPORTED;
   if (dtype == TL_DTYPE_F32)
-    tl::launch_kernel(moe_route_kernel<float>, blocks, ROUTE_WARPS * 32, smem, stream, (const float*)x, ldx, router, choice,
-                      weight, tokens, hidden, experts, top, softmax_scores, renormalize, groups, keep, renorm_eps, correction,
+    tl::launch_kernel(moe_route_kernel<float>, blocks, ROUTE_WARPS * 32, smem, stream, (const float*)x, ldx, router, router_bias, choice,
+                      weight, tokens, hidden, experts, top, score_mode, renormalize, groups, keep, renorm_eps, correction,
                       scale, gate_w, gate_out);
   else
     tl::launch_kernel(moe_route_kernel<__nv_bfloat16>, blocks, ROUTE_WARPS * 32, smem, stream, (const __nv_bfloat16*)x,
-                      ldx, router, choice, weight, tokens, hidden, experts, top, softmax_scores, renormalize, groups, keep,
+                      ldx, router, router_bias, choice, weight, tokens, hidden, experts, top, score_mode, renormalize, groups, keep,
                       renorm_eps, correction, scale, gate_w, gate_out);
   return TL_LAUNCH_CHECK();
 }
@@ -399,23 +418,24 @@ int tl_moe_scatter(const void* x, int ldx, int dtype, const int* position, const
 }
 
 // x [rows, K] sorted rows (rows = max_tiles * 64), w [experts, (2) N, K], out [rows, N].
+// act: 0 none (float32 output), 1 the gated activation over [gate; up], 2 the square of relu (1 and 2: output like x).
 int tl_moe_gemm_simt(const void* x, const void* w, int dtype, void* out, int out_dtype, const int* plan, int max_tiles,
-                     int N, int K, int glu, float limit, float alpha, cudaStream_t stream) {
+                     int N, int K, int act, float limit, float alpha, cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0) return 0;
-  if (K <= 0 || max_tiles > 65535) return TL_ERR_UNSUPPORTED;
+  if (K <= 0 || max_tiles > 65535 || act < 0 || act > 2) return TL_ERR_UNSUPPORTED;
+  if (out_dtype != (act ? dtype : TL_DTYPE_F32)) return TL_ERR_UNSUPPORTED;
   dim3 grid((N + BN - 1) / BN, max_tiles);
-#define TL_MOE(T, OutT, GLU)                                                                                        \
-  tl::launch_kernel(moe_gemm_simt_kernel<T, OutT, GLU>, grid, 256, 0, stream, (const T*)x, (const T*)w, (OutT*)out, \
-                    plan, N, K, limit, alpha)
+#define TL_MOE(T, OutT, GLU, RELU2)                                                                                 \
+  tl::launch_kernel(moe_gemm_simt_kernel<T, OutT, GLU, RELU2>, grid, 256, 0, stream, (const T*)x, (const T*)w,      \
+                    (OutT*)out, plan, N, K, limit, alpha)
   if (dtype == TL_DTYPE_F32) {
-    if (out_dtype != TL_DTYPE_F32) return TL_ERR_UNSUPPORTED;
-    if (glu) TL_MOE(float, float, true); else TL_MOE(float, float, false);
-  } else if (glu) {
-    if (out_dtype != TL_DTYPE_BF16) return TL_ERR_UNSUPPORTED;
-    TL_MOE(__nv_bfloat16, __nv_bfloat16, true);
+    if (act == 1) TL_MOE(float, float, true, false);
+    else if (act == 2) TL_MOE(float, float, false, true);
+    else TL_MOE(float, float, false, false);
   } else {
-    if (out_dtype != TL_DTYPE_F32) return TL_ERR_UNSUPPORTED;
-    TL_MOE(__nv_bfloat16, float, false);
+    if (act == 1) TL_MOE(__nv_bfloat16, __nv_bfloat16, true, false);
+    else if (act == 2) TL_MOE(__nv_bfloat16, __nv_bfloat16, false, true);
+    else TL_MOE(__nv_bfloat16, float, false, false);
   }
 #undef TL_MOE
   return TL_LAUNCH_CHECK();

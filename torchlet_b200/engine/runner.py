@@ -100,6 +100,8 @@ class StepContext:
         self.req_indptr = self.kv_before = self.slots = self.logit_rows = None
         # host copies (numpy int32) for parts that plan on the host
         self.req_indptr_host = self.kv_before_host = self.slots_host = None
+        # what the model itself keeps a slot, by name
+        self.model_state: dict = getattr(getattr(runner, "storage", None), "model_states", {})
         self.plans: dict = {}  # per-step plans parts share across layers
         self._pending: Optional[PendingSum] = None  # see ``leave_pending``
         self._pending_write: Optional[tuple] = None  # see ``leave_write``
@@ -203,7 +205,7 @@ class ModelRunner:
         self.vocab_size = model.spec.vocab_size
         self.storage = CacheStorage(
             model.cache_needs(), config.kv_block_size, config.max_decode_slots, config.max_num_blocks,
-            config.max_seq_len, self.device, self.dtype,
+            config.max_seq_len, self.device, self.dtype, model.state_specs(),
         )
         self.cache = self.storage.manager
         self.num_groups = len(self.storage.groups)
@@ -290,7 +292,7 @@ class ModelRunner:
     def admit(self, request_id: Hashable) -> int:
         slot = self.cache.admit(request_id)
         self._synced.pop(slot, None)
-        if self.storage.states or self.storage.block_states:
+        if self.storage.states or self.storage.block_states or self.storage.model_states:
             self.storage.clear_slot(slot)
         return slot
 

@@ -47,7 +47,7 @@ _SIGNATURES = {
     "attention_generic": {
         "tl_attention_generic": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p,
                                  c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int,
-                                 c_void_p, c_void_p, c_int, c_void_p],
+                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "tl_attention_generic_debug_error": [c_void_p],
     },
     "gemm_tc": {
@@ -155,9 +155,22 @@ _SIGNATURES = {
         "tl_head_finish": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "tl_gated_attention_debug_error": [c_void_p],
     },
+    "qkv_prepare": {
+        "tl_qkv_prepare": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
+                           c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p,
+                           c_int, c_int, c_void_p],
+        "tl_qkv_prepare_debug_error": [c_void_p],
+    },
+    "token_embed": {
+        "tl_token_embed": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                           c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_int,
+                           c_int, c_float, c_void_p],
+        "tl_token_embed_debug_error": [c_void_p],
+    },
     "moe": {
         "tl_moe_tile_rows": [],
-        "tl_moe_route": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+        "tl_moe_route": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_int, c_float, c_void_p, c_float, c_void_p, c_void_p, c_void_p],
         "tl_moe_plan": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "tl_moe_scatter": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -364,8 +377,11 @@ def _sink(sink, nh: int) -> tuple:
 
 
 def attention_generic(q, q_stride, pages, block_table, token_req, positions, out, tokens, nh, nkv, d,
-                      page_size, window, scale, softcap=None, sink=False, gate=None) -> None:
-    """Paged causal GQA attention, one warp per (token, head); q may be a view into qkv.
+                      page_size, window, scale, softcap=None, sink=False, gate=None, keep: int = 0, spread: bool = False,
+                      v_cols=None) -> None:
+    """Paged causal GQA attention, one warp per (token, head); q may be a view into qkv.  ``keep``: the first that many
+    positions stay visible beside the window; ``spread``: query rows span all KV heads, [nh][nkv][d] (``qkv_prepare``);
+    ``v_cols``: value entries a head writes (default d).
     ``softcap``: scores become softcap * tanh(score / softcap); ``sink``: one is added to the softmax's
     denominator (True), or exp(sink[head]) (a float32 tensor [nh]); ``gate`` (float32 [tokens, >= nh * d] rows): the output is multiplied by sigmoid(gate)."""
     _need_cuda(q, pages, block_table, token_req, positions, out, gate)
@@ -375,7 +391,8 @@ def attention_generic(q, q_stride, pages, block_table, token_req, positions, out
         q.data_ptr(), q_stride, pages.data_ptr(), dtype_code(q.dtype), block_table.data_ptr(),
         block_table.shape[1], token_req.data_ptr(), positions.data_ptr(), out.data_ptr(), out.stride(0),
         tokens, nh, nkv, d, page_size, int(window or 0), float(scale), pages.shape[0], float(softcap or 0.0),
-        *_sink(sink, nh), _ptr(gate), gate.stride(0) if gate is not None else 0, _stream())
+        *_sink(sink, nh), _ptr(gate), gate.stride(0) if gate is not None else 0, int(keep), nkv if spread else 1,
+        int(v_cols or d), _stream())
     _check(code, "attention_generic")
 
 
@@ -603,6 +620,66 @@ def normed_qk_store(proj, wq, wk, inv_freq, magnitude: float, eps: float, positi
         1 if wq is not None else 0, 1 if wk is not None else 0, v_offset, 1 if write_kv else 0, _ptr(v_inv_freq),
         v_inv_freq.numel() if v_inv_freq is not None else 0, _stream())
     _check(code, "normed_qk_store")
+
+
+def qkv_prepare(src, sizes: tuple, positions, token_req, req_indptr, block_table, pages, page_size: int, q_out, *, splits=None,
+                row=None, bias=None, wq=None, wk=None, eps: float = 1e-6, inv_freq=None, magnitude: float = 1.0, mix=None, spread: int = 0,
+                v_first=None, value_lambda=None, write_kv: bool = True) -> None:
+    """Float32 projection rows [q (H D) | k (G D) | v (G V)] to queries and cache rows (csrc/qkv_prepare.cu): RMS norm of the
+    whole q and the whole k, rotation of the first ``2 inv_freq.numel()`` entries of every head, value mixing, k and v to
+    the pages padded to P entries, q to ``q_out`` rows.  ``sizes`` = (H, G, D, V, P).  ``splits``: ``src`` holds that many
+    split sums [splits, tokens, row] and ``bias`` (or None) is still to be added.  ``mix`` (float32 [H, H]): the scores of the heads
+    are mixed; ``spread`` 1 writes queries spread over all KV heads ([H][G][P]), 0 the queries themselves ([H][P]), 2 the
+    former for requests with several tokens and the latter for single tokens.  ``v_first`` (float32 [tokens, G V]) without
+    ``value_lambda`` receives this layer's values; with it (a float32 number on the device) v <- (1 - l) v + l v_first."""
+    H, G, D, V, P = sizes
+    _need_cuda(src, positions, token_req, req_indptr, block_table, pages, q_out, bias, wq, wk, inv_freq, mix, v_first, value_lambda)
+    tokens = positions.numel()
+    width = H * D + G * (D + V)
+    assert src.dtype == torch.float32 and pages.is_contiguous() and pages.dtype == q_out.dtype and q_out.stride(1) == 1
+    assert pages.shape[1:] == (2, G, page_size, P) and q_out.shape[0] == tokens
+    if splits is None:
+        assert src.stride(1) == 1 and src.shape[0] == tokens and src.shape[1] >= width and bias is None
+        row = src.stride(0)
+    else:
+        assert src.is_contiguous() and row >= width and (bias is None or bias.numel() == row)
+    for one in (bias, wq, wk, inv_freq, mix, v_first, value_lambda):
+        assert one is None or (one.dtype == torch.float32 and one.is_contiguous())
+    assert mix is None or mix.shape == (H, H)
+    mode = 0 if v_first is None else (1 if value_lambda is None else 2)
+    assert v_first is None or v_first.shape == (tokens, G * V)
+    code = _fn("qkv_prepare", "tl_qkv_prepare")(
+        src.data_ptr(), splits or 1, tokens * row, row, _ptr(bias), _ptr(wq), _ptr(wk), _ptr(inv_freq), float(magnitude),
+        float(eps), positions.data_ptr(), token_req.data_ptr(), req_indptr.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], pages.data_ptr(), dtype_code(q_out.dtype), page_size, pages.shape[0], q_out.data_ptr(),
+        q_out.stride(0), tokens, H, G, D, V, P, 2 * inv_freq.numel() if inv_freq is not None else 0, _ptr(mix), spread,
+        _ptr(v_first), _ptr(value_lambda), mode, 1 if write_kv else 0, _stream())
+    _check(code, "qkv_prepare")
+
+
+def token_embed(table, ids, out, *, scale: float = 1.0, pairs=None, norm=None, ctx_arrays=None, last=None) -> None:
+    """out[t, s] = norm(table[ids[t]] * scale + pair row) for every stream s (csrc/token_embed.cu); out float32 [T, width] or
+    [T, streams, width].  ``pairs`` = (pair table [buckets + 1, width], mul_prev, mul_cur) with ``ctx_arrays`` =
+    (positions, token_req, req_indptr, slots) and ``last`` (int32 [slots]: every request's last token, read and updated).
+    ``norm`` = (weight, bias or None, eps, centre), or None."""
+    pair_table, mul_prev, mul_cur = pairs if pairs is not None else (None, 0, 0)
+    positions, token_req, req_indptr, slots = ctx_arrays if ctx_arrays is not None else (None,) * 4
+    weight, bias, eps, centre = norm if norm is not None else (None, None, 1.0, False)
+    _need_cuda(table, ids, out, pair_table, positions, token_req, req_indptr, slots, last, weight, bias)
+    tokens, width = out.shape[0], out.shape[-1]
+    assert ids.dtype == torch.int32 and out.dtype == torch.float32 and out.is_contiguous() and table.is_contiguous()
+    assert table.shape[1] == width
+    assert pair_table is None or (pair_table.dtype == table.dtype and pair_table.is_contiguous() and pair_table.shape[1] == width
+                                  and last is not None and last.dtype == torch.int32 and last.is_contiguous())
+    for one in (weight, bias):
+        assert one is None or (one.dtype == torch.float32 and one.numel() == width)
+    code = _fn("token_embed", "tl_token_embed")(
+        table.data_ptr(), _ptr(pair_table), dtype_code(table.dtype), ids.data_ptr(), _ptr(positions), _ptr(token_req),
+        _ptr(req_indptr), _ptr(slots), _ptr(last), last.numel() if last is not None else 0,
+        pair_table.shape[0] - 1 if pair_table is not None else 0, mul_prev, mul_cur, _ptr(weight), _ptr(bias), float(eps),
+        1 if centre else 0, out.data_ptr(), tokens, out.shape[1] if out.dim() == 3 else 1, width, table.shape[0], float(scale),
+        _stream())
+    _check(code, "token_embed")
 
 
 def head_finish(rows, positions, v_inv_freq, gate, nh: int, d: int) -> None:
@@ -979,25 +1056,29 @@ def moe_tile_rows() -> int:
 
 
 def moe_route(x, router, choice, weight, softmax_scores: bool = False, renormalize: bool = False, groups: int = 1,
-              keep: int = 1, renorm_eps: float = 0.0, correction=None, scale: float = 1.0, token_gate=None) -> None:
+              keep: int = 1, renorm_eps: float = 0.0, correction=None, scale: float = 1.0, token_gate=None, bias=None,
+              chosen_softmax: bool = False) -> None:
     """choice[t, j], weight[t, j]: the ``top`` experts of every token by score (sigmoid or softmax of the
     float32 router logits) and their scores (csrc/moe.cu), divided by their sum + ``renorm_eps`` if
     ``renormalize``.  ``groups`` > 1: the experts form that many equal groups of neighbours and only experts of the
     ``keep`` groups with the largest best score can be chosen.  ``correction`` (float32 [experts]): the choice goes
     by score + correction, the weights stay the scores.  ``scale`` multiplies the weights.  ``token_gate`` (w float32
     [hidden], out float32 [tokens]): the same kernel also writes out[t] = sigmoid(w . x[t]), the gate of an always-on
-    expert beside the routed ones."""
+    expert beside the routed ones.  ``bias`` (float32 [experts]) is added to the logits.  ``chosen_softmax``: the choice
+    goes by the logits themselves and the weights are the softmax over the chosen ones alone."""
     gate_w, gate_out = token_gate if token_gate is not None else (None, None)
     _need_cuda(x, router, choice, weight, correction, gate_w, gate_out)
     assert gate_w is None or (gate_w.dtype == gate_out.dtype == torch.float32 and gate_w.numel() == x.shape[1]
                               and gate_out.numel() == x.shape[0] and gate_w.is_contiguous() and gate_out.is_contiguous())
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == router.shape[0])
+    assert bias is None or (bias.is_cuda and bias.dtype == torch.float32 and bias.numel() == router.shape[0])
     tokens, hidden = x.shape
     experts, top = router.shape[0], choice.shape[1]
     assert router.dtype == torch.float32 and router.is_contiguous() and router.shape[1] == hidden and x.stride(1) == 1
     assert choice.dtype == torch.int32 and weight.dtype == torch.float32 and choice.is_contiguous() and weight.is_contiguous()
-    code = _fn("moe", "tl_moe_route")(x.data_ptr(), x.stride(0), dtype_code(x.dtype), router.data_ptr(), choice.data_ptr(),
-                                      weight.data_ptr(), tokens, hidden, experts, top, 1 if softmax_scores else 0,
+    code = _fn("moe", "tl_moe_route")(x.data_ptr(), x.stride(0), dtype_code(x.dtype), router.data_ptr(), _ptr(bias),
+                                      choice.data_ptr(), weight.data_ptr(), tokens, hidden, experts, top,
+                                      2 if chosen_softmax else (1 if softmax_scores else 0),
                                       1 if renormalize else 0, int(groups), int(keep), float(renorm_eps), _ptr(correction),
                                       float(scale), _ptr(gate_w), _ptr(gate_out), _stream())
     _check(code, "moe_route")
@@ -1024,16 +1105,18 @@ def moe_scatter(x, position, weight, out, top: int, weighted: bool) -> None:
     _check(code, "moe_scatter")
 
 
-def moe_gemm_simt(x, w, out, plan, glu: bool = False, limit: float = 0.0, alpha: float = 0.0) -> None:
+def moe_gemm_simt(x, w, out, plan, glu: bool = False, limit: float = 0.0, alpha: float = 0.0, relu_squared: bool = False) -> None:
     """Grouped product over expert-sorted rows on CUDA cores: out[r] = W_e(r) x[r]; ``w`` [experts, N, K], or
-    with ``glu`` [experts, 2 N, K] ([gate; up]) and the clamped gated activation applied."""
+    with ``glu`` [experts, 2 N, K] ([gate; up]) and the clamped gated activation applied; ``relu_squared``: the square of
+    relu applied (both activations write rows of x's type)."""
     _need_cuda(x, w, out, plan)
     rows, K = x.shape
     N = out.shape[1]
     assert x.is_contiguous() and w.is_contiguous() and out.is_contiguous() and w.dtype == x.dtype
     assert w.shape[1:] == ((2 if glu else 1) * N, K) and rows == (plan.numel() - 1) * moe_tile_rows() == out.shape[0]
     code = _fn("moe", "tl_moe_gemm_simt")(x.data_ptr(), w.data_ptr(), dtype_code(x.dtype), out.data_ptr(),
-                                          dtype_code(out.dtype), plan.data_ptr(), plan.numel() - 1, N, K, 1 if glu else 0,
+                                          dtype_code(out.dtype), plan.data_ptr(), plan.numel() - 1, N, K,
+                                          1 if glu else (2 if relu_squared else 0),
                                           float(limit), float(alpha), _stream())
     _check(code, "moe_gemm_simt")
 
@@ -1288,13 +1371,13 @@ GROUPED_TILE_ROWS_FEW = 16  # ... and where a group has few rows (the weight-str
 
 
 def gemm_tc_grouped(x, w, out, plan, glu: bool = False, limit: float = 0.0, alpha: float = 0.0,
-                    tile_rows: int = GROUPED_TILE_ROWS) -> None:
+                    tile_rows: int = GROUPED_TILE_ROWS, relu_squared: bool = False) -> None:
     """Grouped product over group-sorted rows on the tcgen05 tensor cores (csrc/gemm_tc.cu with a plan):
     out[r] = W_g(r) x[r].  ``x`` [rows, K] bfloat16 with rows = tile_rows * tiles; ``tile_rows`` 128 (the
     persistent kernel) or 16 (few rows a group: the weight-streaming orientation);
     ``plan`` int32 [1 + tiles] on the device: plan[0] tiles in use, plan[1 + i] the group of row tile i;
     ``w`` [groups, N, K]; ``out`` [rows, N] float32 or bfloat16, or with ``glu`` (``w`` [groups, 2 F, K], gate
-    and up rows interleaved by 16) [rows, F] bfloat16 with the clamped gated activation applied."""
+    and up rows interleaved by 16) [rows, F] bfloat16 with the clamped gated activation applied; ``relu_squared``: bfloat16 rows of max(., 0)^2."""
     _need_cuda(x, w, out, plan)
     _release_workspace()
     rows, K = x.shape
@@ -1305,6 +1388,9 @@ def gemm_tc_grouped(x, w, out, plan, glu: bool = False, limit: float = 0.0, alph
     if glu:
         assert out.dtype == torch.bfloat16
         epilogue = EPI_SWIGLU_BF16
+    elif relu_squared:
+        assert out.dtype == torch.bfloat16
+        epilogue = EPI_RELU2_BF16
     else:
         epilogue = EPI_STORE_BF16 if out.dtype == torch.bfloat16 else EPI_STORE_F32
     code = _fn("gemm_tc", "tl_gemm_tc_grouped")(
@@ -1514,7 +1600,7 @@ def debug_errors() -> list:
     found = []
     for library in ("elementwise", "attention_generic", "attention_mma", "decode_fused", "slots", "stream_ops",
                     "delta_rule", "latent_attention", "latent_attention_mma", "gla", "gated_attention", "hyper",
-                    "pooled_attention", "ssm", "time_mixing", "token_shift"):
+                    "pooled_attention", "ssm", "time_mixing", "token_shift", "qkv_prepare", "token_embed"):
         if any(name in _functions for name in _SIGNATURES[library]):
             value = ctypes.c_int(0)
             code = _fn(library, f"tl_{library}_debug_error")(ctypes.byref(value))

@@ -38,15 +38,17 @@ class KVSpec:
     """Per-token history a mixer keeps in pages: keys and values of every token,
     or of the last ``window`` tokens only.  ``planes`` is how many rows of ``head_dim`` a token
     keeps per KV head: 2 (a key and a value), or 1 for a mixer whose keys and values are
-    expanded from one cached row (a latent)."""
+    expanded from one cached row (a latent).  ``keep_first``: beside the window, the first that many
+    tokens of a sequence stay (their pages are never given back while the request lives)."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     planes: int = 2
+    keep_first: int = 0
 
     def group_key(self) -> tuple:
-        return (self.num_kv_heads, self.head_dim, self.window, self.planes)
+        return (self.num_kv_heads, self.head_dim, self.window, self.planes, self.keep_first if self.window is not None else 0)
 
 
 @dataclass(frozen=True)

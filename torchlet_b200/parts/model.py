@@ -41,6 +41,8 @@ def _layer_parts(layer) -> list:
 def expected_tensors(spec: ModelSpec) -> list[TensorSpec]:
     """Every tensor the checkpoint must hold, by name, with its shape."""
     out = [TensorSpec(spec.embedding_name, (spec.vocab_size, spec.hidden_size))]
+    if spec.token_pairs is not None:
+        out.append(TensorSpec(spec.token_pairs.table_name, (spec.token_pairs.buckets + 1, spec.hidden_size)))
     if spec.stream_rows_name is not None:
         out.append(TensorSpec(spec.stream_rows_name, (spec.stream_rows, spec.hidden_size)))
     if spec.embedding_norm is not None:
@@ -81,6 +83,7 @@ class LayeredModel:
         self.final_norm = build_part(NORMS, spec.final_norm)
         self.embedding_norm = build_part(NORMS, spec.embedding_norm) if spec.embedding_norm is not None else None
         self.embedding: torch.Tensor | None = None
+        self.pair_table: torch.Tensor | None = None  # [buckets + 1, hidden], see ``TokenPairs``
         self.stream_rows: torch.Tensor | None = None  # [rows, hidden] float32, see ``ScheduleEntry.add_row``
         self.lm_head: Linear | None = None
         self.dtype: torch.dtype | None = None
@@ -101,12 +104,18 @@ class LayeredModel:
                                             self.blocks[entry.layer].state_spec()))
         return needs
 
+    def state_specs(self) -> dict:
+        """What the model itself keeps per live request (name -> ``StateSpec``; ``ctx.model_state`` holds the tensors)."""
+        return {"last_token": StateSpec((1,), "int32")} if self.spec.token_pairs is not None else {}
+
     # --------------------------------------------------------------- weights
     def load(self, tensors: dict, device, dtype: torch.dtype) -> None:
         """Lay the checkpoint's tensors (by name) out on the device for the kernels."""
         spec = self.spec
         self.device, self.dtype = torch.device(device), dtype
         self.embedding = tensors[spec.embedding_name].to(device=device, dtype=dtype).contiguous()
+        if spec.token_pairs is not None:
+            self.pair_table = tensors[spec.token_pairs.table_name].to(device=device, dtype=dtype).contiguous()
         if spec.stream_rows_name is not None:
             self.stream_rows = tensors[spec.stream_rows_name].to(device=device, dtype=torch.float32).contiguous()
         for layer, block in zip(spec.layers, self.blocks):
@@ -128,19 +137,20 @@ class LayeredModel:
         """Run the step's tokens through the schedule; returns the float32 stream [T, hidden]."""
         shape = (ctx.num_tokens, self.spec.hidden_size)
         acc = ctx.buffer("stream", shape, torch.float32)
+        streams = self.spec.streams
+        z = None
+        if streams is not None:
+            z = ctx.buffer("streams", (ctx.num_tokens, streams, self.spec.hidden_size), torch.float32)
         again = any(entry.add_embedding for entry in self.spec.schedule)
         first = ctx.buffer("stream.first", shape, torch.float32) if again else None  # the embedding output, kept
-        if self.embedding_norm is None:
-            ops.embed(self.embedding, ctx.tokens, acc, self.spec.embedding_scale)
+        if self._embeds_at_once():
+            self._embed_at_once(ctx, acc if streams is None else z)
             if again:
-                ops.embed(self.embedding, ctx.tokens, first, self.spec.embedding_scale)
-        else:  # the norm writes float32 rows: the stream stays 32-bit from its first value on
-            raw = ctx.buffer("stream.embedding", shape, torch.float32)
-            ops.embed(self.embedding, ctx.tokens, raw, self.spec.embedding_scale)
-            self.embedding_norm.apply(ctx, raw, out=acc)
-            if again:
-                self.embedding_norm.apply(ctx, raw, out=first)
-        streams = self.spec.streams
+                first.copy_(acc)
+        else:
+            self._embed(ctx, acc, first)
+            if streams is not None:
+                ops.hyper_fanout(acc, z)
         if streams is None:
             for i, entry in enumerate(self.spec.schedule):
                 if entry.add_embedding:
@@ -152,13 +162,41 @@ class LayeredModel:
             ctx.flush_pending()
             return acc
         # several residual streams a token, all equal to the embedding at the start; their sum at the end
-        z = ctx.buffer("streams", (ctx.num_tokens, streams, self.spec.hidden_size), torch.float32)
-        ops.hyper_fanout(acc, z)
         for i, entry in enumerate(self.spec.schedule):
             self.blocks[entry.layer].forward(ctx, z, caches[i])
         ctx.flush_pending()
         ops.hyper_collapse(z, acc)
         return acc
+
+    def _embeds_at_once(self) -> bool:
+        """Whether token row, pair row, norm and the copies to the streams run as one kernel: a model with a pair table
+        (its norm, if it has one, must be over whole rows)."""
+        if self.spec.token_pairs is None:
+            return False
+        if self.embedding_norm is not None and self.embedding_norm.residual_terms() is None:
+            raise ValueError("a table of token pairs is not built together with a grouped norm of the embedding")
+        return True
+
+    def _embed_at_once(self, ctx, out) -> None:
+        pairs = self.spec.token_pairs
+        norm = self.embedding_norm.residual_terms() if self.embedding_norm is not None else None
+        ops.token_embed(self.embedding, ctx.tokens, out, scale=self.spec.embedding_scale,
+                        pairs=(self.pair_table, pairs.mul_prev, pairs.mul_cur), norm=norm,
+                        ctx_arrays=(ctx.positions, ctx.token_req, ctx.req_indptr, ctx.slots), last=ctx.model_state["last_token"])
+
+    def _embed(self, ctx, acc, first) -> None:
+        """The embedding output into ``acc`` (and into ``first``, if that is kept)."""
+        if self.embedding_norm is None:
+            ops.embed(self.embedding, ctx.tokens, acc, self.spec.embedding_scale)
+            if first is not None:
+                ops.embed(self.embedding, ctx.tokens, first, self.spec.embedding_scale)
+            return
+        # the norm writes float32 rows: the stream stays 32-bit from its first value on
+        raw = ctx.buffer("stream.embedding", tuple(acc.shape), torch.float32)
+        ops.embed(self.embedding, ctx.tokens, raw, self.spec.embedding_scale)
+        self.embedding_norm.apply(ctx, raw, out=acc)
+        if first is not None:
+            self.embedding_norm.apply(ctx, raw, out=first)
 
     def logits(self, ctx, acc: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
         """Float32 logits of the stream rows ``rows`` (int32) into ``out`` [len(rows), vocab]."""

@@ -1,6 +1,7 @@
 """A routed feed-forward (mixture of experts) of gated units, clamped or plain.
 
-Router: z = W_router x in float32, scores sigmoid(z) (``score`` "sigmoid") or softmax(z) ("softmax");
+Router: z = W_router x (+ b_router with ``router_bias``) in float32, scores sigmoid(z) (``score`` "sigmoid") or softmax(z)
+("softmax"), or the logits themselves, whose chosen ones the weights are the softmax over ("chosen_softmax");
 every token uses the ``top_k`` experts with the largest scores (the lower index wins a tie); the
 weights are those scores, divided by their sum if ``renormalize``.  Expert e: g = min(W_gate,e h, limit),
 u = clamp(W_up,e h, -limit, limit), y = g sigmoid(alpha g) (u + 1), output W_down,e y, no biases.  The
@@ -12,6 +13,8 @@ can be chosen.  With ``renormalize`` the chosen scores are divided by their sum 
 ``correction``: a tensor of one number an expert is added to the scores for the CHOICE only (the weights stay the
 scores).  ``weight_scale`` multiplies the weights.  ``identity`` = n: the router has n more outputs than there are
 experts; the last n are identity experts without tensors, whose output is their input (times the weight).
+``unit`` "relu_squared": the experts are ungated, W_down,e max(W_up,e h, 0)^2, without gate tensors ("glu", the default:
+the gated unit above).
 ``shared``: a feed-forward part (with its prefix ``shared_prefix`` below this one's) that runs for every token beside
 the routed experts and adds its own output.
 
@@ -24,8 +27,8 @@ kernel does not take, on CUDA cores in tiles of 64 rows.
 
 Parameters: ``hidden_size``, ``intermediate_size``, ``limit``, ``alpha``, ``num_experts``, ``top_k``,
 ``score``, ``renormalize``, ``renorm_eps``, ``weight_on``, ``groups``, ``keep``, ``correction``, ``weight_scale``,
-``identity``, ``shared``, ``shared_prefix``.  Tensors below the prefix: router [E + identity, hidden];
-e<j>.gate, e<j>.up [ff, hidden]; e<j>.down [hidden, ff]; correction [E + identity].
+``identity``, ``shared``, ``shared_prefix``, ``unit``, ``router_bias``.  Tensors below the prefix: router [E + identity, hidden];
+e<j>.gate, e<j>.up [ff, hidden]; e<j>.down [hidden, ff]; correction [E + identity]; router.b [E + identity].
 """
 from __future__ import annotations
 
@@ -59,8 +62,13 @@ class RoutedClampedGLU(FeedForward):
             raise ValueError(f"{self.num_experts} experts cannot form {self.groups} equal groups of which {self.keep} are kept")
         if self.top_k > self.keep * ((self.num_experts + int(p.get("identity", 0) or 0)) // self.groups):
             raise ValueError(f"top_k {self.top_k} exceeds the {self.keep} kept groups' experts")
-        if self.score not in ("sigmoid", "softmax"):
-            raise ValueError(f"unknown router score {self.score!r} (known: sigmoid, softmax)")
+        if self.score not in ("sigmoid", "softmax", "chosen_softmax"):
+            raise ValueError(f"unknown router score {self.score!r} (known: sigmoid, softmax, chosen_softmax)")
+        self.unit = p.get("unit", "glu")
+        if self.unit not in ("glu", "relu_squared"):
+            raise ValueError(f"unknown expert unit {self.unit!r} (known: glu, relu_squared)")
+        self.has_router_bias = bool(p.get("router_bias", False))
+        self.router_bias = None
         if self.weight_on not in ("input", "output"):
             raise ValueError(f"weight_on must be 'input' or 'output', got {self.weight_on!r}")
         if not 0 < self.top_k <= self.num_experts + int(p.get("identity", 0) or 0):
@@ -78,7 +86,7 @@ class RoutedClampedGLU(FeedForward):
         self.shared = build_part(FEED_FORWARDS, p["shared"]) if p.get("shared") is not None else None
         self.shared_prefix = str(p.get("shared_prefix", "shared."))
         self.correction = None
-        self.router = self.gate_up = self.down = None
+        self.router = self.gate_up = self.down = None  # gate_up: the first product's weights (of an ungated expert: up alone)
         self.tensor_cores = False
 
     @classmethod
@@ -87,10 +95,13 @@ class RoutedClampedGLU(FeedForward):
         hidden, inter, experts = int(p["hidden_size"]), int(p["intermediate_size"]), int(p["num_experts"])
         out = []
         for e in range(experts):
-            out += [TensorSpec(f"{prefix}e{e}.gate", (inter, hidden)), TensorSpec(f"{prefix}e{e}.up", (inter, hidden)),
-                    TensorSpec(f"{prefix}e{e}.down", (hidden, inter))]
+            if p.get("unit", "glu") == "glu":
+                out.append(TensorSpec(f"{prefix}e{e}.gate", (inter, hidden)))
+            out += [TensorSpec(f"{prefix}e{e}.up", (inter, hidden)), TensorSpec(f"{prefix}e{e}.down", (hidden, inter))]
         outputs = experts + int(p.get("identity", 0) or 0)
         out.append(TensorSpec(prefix + "router", (outputs, hidden)))
+        if p.get("router_bias", False):
+            out.append(TensorSpec(prefix + "router.b", (outputs,), init="zeros"))
         if p.get("correction", False):
             out.append(TensorSpec(prefix + "correction", (outputs,), init="zeros"))
         if p.get("shared") is not None:
@@ -100,6 +111,8 @@ class RoutedClampedGLU(FeedForward):
     def load(self, tensors: dict, prefix: str, device, dtype) -> None:
         E = self.num_experts
         self.router = tensors[prefix + "router"].to(device=device, dtype=torch.float32).contiguous()
+        if self.has_router_bias:
+            self.router_bias = tensors[prefix + "router.b"].to(device=device, dtype=torch.float32).contiguous()
         if self.has_correction:
             self.correction = tensors[prefix + "correction"].to(device=device, dtype=torch.float32).contiguous()
         if self.shared is not None:
@@ -110,9 +123,13 @@ class RoutedClampedGLU(FeedForward):
         # gate and up rows of an expert are interleaved by 16 instead, as the gated epilogue reads them
         self.tensor_cores = (dtype == torch.bfloat16 and swiglu_bf16.usable(self.hidden_size, self.intermediate_size)
                              and self.intermediate_size % 8 == 0)
-        join = swiglu_bf16.interleave if self.tensor_cores else (lambda gate, up: torch.cat([gate, up], dim=0))
-        self.gate_up = torch.stack([join(tensors[f"{prefix}e{e}.gate"], tensors[f"{prefix}e{e}.up"])
-                                    for e in range(E)]).to(device=device, dtype=dtype).contiguous()
+        if self.unit == "relu_squared":
+            self.tensor_cores = dtype == torch.bfloat16 and self.hidden_size % 8 == 0 and self.intermediate_size % 8 == 0
+            rows = [tensors[f"{prefix}e{e}.up"] for e in range(E)]
+        else:
+            join = swiglu_bf16.interleave if self.tensor_cores else (lambda gate, up: torch.cat([gate, up], dim=0))
+            rows = [join(tensors[f"{prefix}e{e}.gate"], tensors[f"{prefix}e{e}.up"]) for e in range(E)]
+        self.gate_up = torch.stack(rows).to(device=device, dtype=dtype).contiguous()
         self.down = torch.stack([tensors[f"{prefix}e{e}.down"] for e in range(E)]).to(device=device, dtype=dtype).contiguous()
 
     def _rows(self, tokens: int, tile: int) -> tuple:
@@ -151,15 +168,16 @@ class RoutedClampedGLU(FeedForward):
         shared_gate = ctx.buffer("moe.shared_gate", (tokens,), torch.float32) if gate_w is not None else None
         ops.moe_route(x, self.router, choice, weight, self.score == "softmax", self.renormalize, self.groups, self.keep,
                       self.renorm_eps, correction=self.correction, scale=self.weight_scale,
-                      token_gate=(gate_w, shared_gate) if gate_w is not None else None)
+                      token_gate=(gate_w, shared_gate) if gate_w is not None else None, bias=self.router_bias,
+                      chosen_softmax=self.score == "chosen_softmax")
         ops.moe_plan(choice, position, plan, E, tile)
         ops.moe_scatter(x, position, weight, sorted_x, top, weighted=on_input)
+        unit = {"relu_squared": True} if self.unit == "relu_squared" else {"glu": True, "limit": self.limit, "alpha": self.alpha}
         if self.tensor_cores:
-            ops.gemm_tc_grouped(sorted_x, self.gate_up, act, plan, glu=True, limit=self.limit, alpha=self.alpha,
-                                tile_rows=tile)
+            ops.gemm_tc_grouped(sorted_x, self.gate_up, act, plan, tile_rows=tile, **unit)
             ops.gemm_tc_grouped(act, self.down, y, plan, tile_rows=tile)
         else:
-            ops.moe_gemm_simt(sorted_x, self.gate_up, act, plan, glu=True, limit=self.limit, alpha=self.alpha)
+            ops.moe_gemm_simt(sorted_x, self.gate_up, act, plan, **unit)
             ops.moe_gemm_simt(act, self.down, y, plan)
         ops.moe_combine(y, position, weight, acc, top, weighted=not on_input, x=x if self.identity else None)
         if self.shared is not None and shared_gate is not None:
