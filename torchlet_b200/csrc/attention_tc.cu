@@ -202,7 +202,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) 
   uint64_t* s_full = bars + 8;    // [2 row tiles]  S_X of the next key tile is in tensor memory
   uint64_t* p_full = bars + 10;   // [2 row tiles]  (4 arrivals: one per softmax warp) P_X is written
   uint64_t* o_done = bars + 12;   // [2 row tiles]  the last P_X V is done
-  uint64_t* v_clean = bars + 14;  // value rows outside the CTA's keys are cleared (edge tiles only)
+  uint64_t* v_clean = bars + 14;  // [2: the CTA's first key tile, its last] value rows outside its keys are cleared
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
@@ -266,7 +266,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) 
       mbar_init(&p_full[i], 4);
       mbar_init(&o_done[i], 1);
     }
-    mbar_init(v_clean, 1);
+    mbar_init(&v_clean[0], 1);
+    mbar_init(&v_clean[1], 1);
     *abort_flag = 0;
     mbar_fence_init();
     prefetch_tensormap(&map_kv);
@@ -333,7 +334,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) 
         }
         fence_proxy_async();  // the tensor core reads, and later copies overwrite, what these stores wrote
         __syncwarp();
-        if (lane == 0) mbar_arrive(v_clean);
+        if (lane == 0) mbar_arrive(&v_clean[j == j_begin && edge_first ? 0 : 1]);
       }
     }
   } else if (warp == 8) {
@@ -358,8 +359,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const Params p) 
       // V of the previous key tile has long arrived, K of this one nearly always
       if (jj > 0) mbar_wait(&v_full[(jj - 1) & 1], ((jj - 1) >> 1) & 1, abort_flag, &g_error_word, 6);
       if (jj > 0 && ((edge_first && j - 1 == j_begin) || (edge_last && j == j_end)))
-        mbar_wait(v_clean, (edge_first && edge_last && j == j_end && j_end - j_begin > 1) ? 1 : 0, abort_flag,
-                  &g_error_word, 11);
+        mbar_wait(&v_clean[edge_first && j - 1 == j_begin ? 0 : 1], 0, abort_flag, &g_error_word, 11);
       if (j < j_end) mbar_wait(&k_full[jj & 1], (jj >> 1) & 1, abort_flag, &g_error_word, 3);
       // the last row tile with work at this step (row tile 0 always has some)
       const bool work_1 = (j - 1 >= tile[1].begin && j - 1 < tile[1].end) || (j >= tile[1].begin && j < tile[1].end);

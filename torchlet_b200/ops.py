@@ -92,6 +92,21 @@ _SIGNATURES = {
         "tl_attention_tc_error": [],
         "tl_attention_tc_rows": [c_int],
     },
+    "attention_spread": {
+        "tl_attention_spread": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                c_int, c_float, c_void_p],
+        "tl_attention_spread_rows": [c_int],
+        "tl_attention_spread_error": [],
+    },
+    "attention_mixed_decode": {
+        "tl_attention_mixed_decode": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                      c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                      c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p],
+        "tl_attention_mixed_decode_tile": [c_int, c_int, c_int, c_int, c_int],
+        "tl_attention_mixed_decode_error": [],
+        "tl_attention_mixed_decode_debug_error": [c_void_p],
+    },
     "slots": {
         "tl_slot_gather": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -1574,6 +1589,73 @@ def attention_tc(qkv, pages, block_table, req_indptr, kv_before, tile_req, tile_
     return merge
 
 
+def attention_spread_rows(group: int) -> int:
+    """Packed rows a tile of the prompt kernel for mixed scores holds for ``group`` heads a KV head."""
+    return _fn("attention_spread", "tl_attention_spread_rows")(group)
+
+
+def attention_spread_supported(p_size: int, group: int, page_size: int, scale: float) -> bool:
+    return p_size in (64, 128) and 1 <= group <= 128 and 8 <= page_size <= 128 and 128 % page_size == 0 and scale > 0
+
+
+def attention_spread(q, pages, block_table, req_indptr, kv_before, tile_req, tile_row, tiles, out, *, nh, nkv, p_size,
+                     page_size, window, keep, v_cols, scale, spread: bool) -> None:
+    """Prompt-portion attention on tcgen05 (csrc/attention_spread.cu): a window beside which the first ``keep`` tokens stay
+    visible, and, with ``spread``, query rows [nh][nkv][p_size] whose score with a token is their dot product with all of its
+    keys (``qkv_prepare``); without it rows [nh][p_size] against the head's own KV head.  ``tile_row``: multiples of
+    ``attention_spread_rows(nh // nkv)``.  out [tokens, nh v_cols]."""
+    _need_cuda(q, pages, block_table, req_indptr, kv_before, tile_req, tile_row, out)
+    assert q.dtype == pages.dtype == out.dtype == torch.bfloat16 and pages.is_contiguous() and out.stride(1) == 1
+    assert q.shape[1] >= nh * p_size * (nkv if spread else 1) and out.shape[1] == nh * v_cols
+    code = _fn("attention_spread", "tl_attention_spread")(
+        q.data_ptr(), q.stride(0), pages.data_ptr(), pages.shape[0], block_table.data_ptr(), block_table.shape[1],
+        req_indptr.data_ptr(), kv_before.data_ptr(), tile_req.data_ptr(), tile_row.data_ptr(), tiles, out.data_ptr(),
+        out.stride(0), q.shape[0], nh, nkv, p_size, page_size, int(window or 0), int(keep), nkv if spread else 1, v_cols,
+        float(scale), _stream())
+    _check(code, "attention_spread")
+
+
+def attention_mixed_decode_tile(nh: int, nkv: int, p_size: int, page_size: int, v_cols: int) -> int:
+    """Keys a tile of the single-token kernel for mixed scores holds; 0: it does not take these sizes."""
+    return _fn("attention_mixed_decode", "tl_attention_mixed_decode_tile")(nh, nkv, p_size, page_size, v_cols)
+
+
+def attention_mixed_decode(q, pages, block_table, req_indptr, kv_before, tile_req, tiles, out, *, nh, nkv, p_size, page_size,
+                           window, keep, v_cols, scale, talk=None, splits: int = 1) -> None:
+    """Single-token attention that computes all heads' scores of a key at once (csrc/attention_mixed_decode.cu) and mixes
+    them with ``talk`` (float32 [nh, nh]; None: no mixing).  q rows begin with [nh][p_size]; ``tile_req``: the requests that
+    bring one token (None: all).  ``splits``: CTAs the grid holds for a request's keys; it uses as many as its length
+    warrants.  Only those tokens' rows of ``out`` [tokens, nh v_cols] are written."""
+    _need_cuda(q, pages, block_table, req_indptr, kv_before, tile_req, out, talk)
+    assert q.dtype == pages.dtype == out.dtype == torch.bfloat16 and pages.is_contiguous() and out.stride(1) == 1
+    assert out.shape[1] == nh * v_cols and q.shape[1] >= nh * p_size
+    assert talk is None or (talk.dtype == torch.float32 and talk.is_contiguous() and talk.shape == (nh, nh))
+    need = tiles * splits * nh * (p_size + 2) * 4 if splits > 1 else 0
+    ws = _workspace(("attention", q.device), need) if need else None
+    arrivals = _arrivals(q.device, tiles) if need else None
+    code = _fn("attention_mixed_decode", "tl_attention_mixed_decode")(
+        q.data_ptr(), q.stride(0), pages.data_ptr(), pages.shape[0], block_table.data_ptr(), block_table.shape[1],
+        req_indptr.data_ptr(), kv_before.data_ptr(), _ptr(tile_req), tiles, out.data_ptr(), out.stride(0), nh, nkv, p_size,
+        page_size, int(window or 0), int(keep), v_cols, float(scale), _ptr(talk), splits, _ptr(ws),
+        ws.numel() * 4 if ws is not None else 0, _ptr(arrivals), _stream())
+    _check(code, "attention_mixed_decode")
+
+
+def attention_mixed_decode_error() -> int:
+    """0, or the code a bounded wait of the single-token kernel for mixed scores left.  Reading clears it (and the arrival
+    counters)."""
+    code = _fn("attention_mixed_decode", "tl_attention_mixed_decode_error")()
+    if code:
+        for counters in _arrival_counters.values():
+            counters.zero_()
+    return code
+
+
+def attention_spread_error() -> int:
+    """0, or the code a bounded wait in the prompt kernel for mixed scores left when it gave up."""
+    return _fn("attention_spread", "tl_attention_spread_error")()
+
+
 def attention_mma_error() -> int:
     """0, or the code a bounded wait of the decode attention's TMA loader left.  Reading clears it
     (and the arrival counters, which a kernel that gave up may have left half counted)."""
@@ -1600,7 +1682,8 @@ def debug_errors() -> list:
     found = []
     for library in ("elementwise", "attention_generic", "attention_mma", "decode_fused", "slots", "stream_ops",
                     "delta_rule", "latent_attention", "latent_attention_mma", "gla", "gated_attention", "hyper",
-                    "pooled_attention", "ssm", "time_mixing", "token_shift", "qkv_prepare", "token_embed"):
+                    "pooled_attention", "ssm", "time_mixing", "token_shift", "qkv_prepare", "token_embed",
+                    "attention_mixed_decode"):
         if any(name in _functions for name in _SIGNATURES[library]):
             value = ctypes.c_int(0)
             code = _fn(library, f"tl_{library}_debug_error")(ctypes.byref(value))
@@ -1616,7 +1699,8 @@ def raise_on_wait_errors() -> None:
     Only libraries that are loaded are asked.  The read is a blocking copy on the default
     stream, so it sees every kernel launched before it."""
     for library, read in (("gemm_tc", gemm_tc_error), ("attention_tc", attention_tc_error),
-                          ("attention_mma", attention_mma_error)):
+                          ("attention_mma", attention_mma_error), ("attention_spread", attention_spread_error),
+                          ("attention_mixed_decode", attention_mixed_decode_error)):
         if any(name in _functions for name in _SIGNATURES[library]):
             code = read()
             if code:

@@ -272,7 +272,7 @@ class GatedAttentionMixer(Mixer):
             magnitude=positions.magnitude if positions is not None else 1.0, mix=self.talk, spread=spread, v_first=v_first,
             value_lambda=self.value_lambda, write_kv=cache.writable, **source)
         out = ctx.buffer("gated_attention.out", (tokens, H * self.v_dim), ctx.dtype)
-        if not mixed_attention_bf16.forward(self, ctx, q, cache, out, spread):
+        if not mixed_attention_bf16.forward(self, ctx, q, cache, out):
             ops.attention_generic(q, q.stride(0), cache.pages, cache.block_table, ctx.token_req, ctx.positions, out, tokens,
                                   H, G, self.head_dim, cache.page_size, self.window, self.scale, keep=self.keep_first,
                                   spread=bool(spread), v_cols=self.v_dim)
