@@ -53,7 +53,7 @@ def designed(T, H, G, P, V, window, keep, at, td, seed=0):
 SIZES = [  # H, G, P, V, window, keep, page size
     (4, 2, 64, 64, 40, 5, 16), (8, 8, 64, 24, 64, 64, 8), (16, 4, 128, 128, 100, 1, 16), (6, 1, 128, 96, 129, 140, 32),
     (16, 1, 64, 64, 1, 17, 16), (32, 8, 128, 128, 70, 30, 64), (12, 3, 128, 33, 33, 0, 16), (20, 10, 64, 64, 250, 20, 128),
-    (5, 5, 64, 48, None, 0, 16), (24, 2, 64, 64, 128, 128, 8)]
+    (5, 5, 64, 48, None, 0, 16), (24, 2, 64, 64, 128, 128, 8), (64, 8, 128, 128, 60, 25, 16)]
 
 
 @pytest.mark.parametrize("H,G,P,V,window,keep,page_size", SIZES)

@@ -23,8 +23,6 @@ namespace {
 
 using namespace tl;
 
-constexpr int NT = 256;
-
 struct Params {
   const float* src;  // [splits][tokens][src_stride]
   int splits;
@@ -36,6 +34,7 @@ struct Params {
   int table_width, page_size, num_pages;
   int H, G, D, V, P, dims;
   const float* mix;  // [H][H] or null
+  int mix_floats;    // shared memory it takes
   int spread;
   float* v_first;  // [tokens][G V]
   const float* lambda;
@@ -44,120 +43,210 @@ struct Params {
   long long q_stride;
 };
 
-template <typename T> __device__ __forceinline__ void store2(T* p, float a, float b);
-template <> __device__ __forceinline__ void store2<float>(float* p, float a, float b) {
-  *reinterpret_cast<float2*>(p) = make_float2(a, b);
+// W consecutive floats (4 where every size and address allows 16-byte pieces, else 1).
+template <int W> __device__ __forceinline__ void load_w(const float* p, float (&v)[W]) {
+  if constexpr (W == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+  } else {
+    v[0] = *p;
+  }
 }
-template <> __device__ __forceinline__ void store2<__nv_bfloat16>(__nv_bfloat16* p, float a, float b) {
-  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+template <int W> __device__ __forceinline__ void store_w(float* p, const float (&v)[W]) {
+  if constexpr (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+template <int W> __device__ __forceinline__ void store_w(__nv_bfloat16* p, const float (&v)[W]) {
+  if constexpr (W == 4) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+  } else {
+    *p = __float2bfloat16_rn(v[0]);
+  }
 }
 
 // q' of one token; ``PER`` = H / G query heads a KV head where that is 1, 2, 4 or 8 (their entries then stay in
 // registers for all H rows), else 0.
-template <typename T, int PER>
+template <typename T, int NT, int PER, int W>
 __device__ __forceinline__ void spread_queries(const Params& p, const float* q, const float* mix, T* out) {
   const int per = PER > 0 ? PER : p.H / p.G;
-  const int pairs = p.P >> 1, items = p.G * pairs;
-  const int rows = max(1, min(p.H, NT / max(1, items)));  // threads that share a column pair, each with its own heads
+  const int pieces = p.P / W, items = p.G * pieces;
+  const int rows = max(1, min(p.H, NT / max(1, items)));  // threads that share a column piece, each with its own heads
   for (int item = threadIdx.x; item < items * rows; item += NT) {
-    const int col = item % items, part = item / items;
-    const int c = col / pairs, i = (col - c * pairs) * 2;
-    const bool in0 = i < p.D, in1 = i + 1 < p.D;
-    const float* base = q + (size_t)c * per * p.D + i;
-    float v0[PER > 0 ? PER : 1], v1[PER > 0 ? PER : 1];
+    const int part = item / items, col = item - part * items;
+    const int c = col / pieces, i = (col - c * pieces) * W;
+    const bool in = i < p.D;
+    const float* base = q + (size_t)c * per * p.D + (in ? i : 0);
+    float v[PER > 0 ? PER : 1][W];
     if constexpr (PER > 0) {
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
-        v0[j] = in0 ? base[j * p.D] : 0.f;
-        v1[j] = in1 ? base[j * p.D + 1] : 0.f;
+        load_w<W>(base + j * p.D, v[j]);
+        if (!in)
+#pragma unroll
+          for (int e = 0; e < W; ++e) v[j][e] = 0.f;
       }
     }
     for (int h = part; h < p.H; h += rows) {
       const float* m = mix + h * p.H + c * per;
-      float a = 0.f, b = 0.f;
-      if constexpr (PER > 0) {
+      float sum[W];
 #pragma unroll
-        for (int j = 0; j < PER; ++j) {
-          a = fmaf(m[j], v0[j], a);
-          b = fmaf(m[j], v1[j], b);
+      for (int e = 0; e < W; ++e) sum[e] = 0.f;
+      if constexpr (PER > 0) {
+        float f[PER];
+        if constexpr (PER % 4 == 0) {  // (rows of the matrix then start on 16-byte boundaries)
+#pragma unroll
+          for (int j = 0; j < PER; j += 4) load_w<4>(m + j, reinterpret_cast<float(&)[4]>(f[j]));
+        } else {
+#pragma unroll
+          for (int j = 0; j < PER; ++j) f[j] = m[j];
         }
-      } else {
+#pragma unroll
+        for (int j = 0; j < PER; ++j)
+#pragma unroll
+          for (int e = 0; e < W; ++e) sum[e] = fmaf(f[j], v[j][e], sum[e]);
+      } else if (in) {
         for (int j = 0; j < per; ++j) {
-          a = fmaf(m[j], in0 ? base[j * p.D] : 0.f, a);
-          b = fmaf(m[j], in1 ? base[j * p.D + 1] : 0.f, b);
+          float one[W];
+          load_w<W>(base + j * p.D, one);
+#pragma unroll
+          for (int e = 0; e < W; ++e) sum[e] = fmaf(m[j], one[e], sum[e]);
         }
       }
-      store2<T>(out + ((size_t)h * p.G + c) * p.P + i, a, b);
+      store_w<W>(out + ((size_t)h * p.G + c) * p.P + i, sum);
     }
   }
 }
 
-template <typename T>
+// NT threads a token: 256, or 1,024 for a few tokens whose product left split sums (a thread then walks one piece).
+template <typename T, int NT, int W>
 __global__ void __launch_bounds__(NT)
 qkv_prepare_kernel(const Params p, T* __restrict__ pages, T* __restrict__ q_out) {
   tl::pdl_launch_dependents();
-  tl::pdl_wait();
   extern __shared__ __align__(16) float smem[];
   __shared__ float scratch[32];
   const int t = blockIdx.x;
   const int qn = p.H * p.D, kn = p.G * p.D, vn = p.G * p.V, half = p.dims >> 1;
-  float* q = smem;            // H D
-  float* k = q + qn;          // G D
-  float* v = k + kn;          // G V
-  float* cosines = v + vn;    // half
-  float* sines = cosines + half;
-  float* mix = sines + half;  // H H
+  float* mix = smem;                         // H H (rounded up to a multiple of 4)
+  float* q = mix + p.mix_floats;             // H D
+  float* k = q + qn;                         // G D
+  float* v = k + kn;                         // G V
+  float* cosines = v + (vn + 3) / 4 * 4;     // half
+  float* sines = cosines + (half + 3) / 4 * 4;
+  if (p.mix_floats && p.spread)  // weights: before the wait
+    for (int i = threadIdx.x; i < p.H * p.H; i += NT) mix[i] = p.mix[i];
+  tl::pdl_wait();
   const int pos = p.positions[t];
   const int req = p.token_req[t];
   const bool spread = p.mix && (p.spread == 1 || (p.spread == 2 && p.req_indptr[req + 1] - p.req_indptr[req] > 1));
+  const float* row = p.src + (size_t)t * p.src_stride;
+  float ssq = 0.f, ssk = 0.f;
+  for (int i = threadIdx.x * W; i < qn + kn + vn; i += NT * W) {
+    float x[W];
+    if (p.splits == 1) {
+      load_w<W>(row + i, x);
+    } else {  // ascending splits, eight loads in flight
+#pragma unroll
+      for (int e = 0; e < W; ++e) x[e] = 0.f;
+      for (int s = 0; s < p.splits; s += 8) {
+        float one[8][W];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (s + j < p.splits) load_w<W>(row + (size_t)(s + j) * p.split_stride + i, one[j]);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (s + j < p.splits)
+#pragma unroll
+            for (int e = 0; e < W; ++e) x[e] += one[j][e];
+      }
+    }
+    if (p.bias) {
+      float b[W];
+      load_w<W>(p.bias + i, b);
+#pragma unroll
+      for (int e = 0; e < W; ++e) x[e] += b[e];
+    }
+    store_w<W>(q + i, x);
+#pragma unroll
+    for (int e = 0; e < W; ++e) {
+      if (i < qn) ssq = fmaf(x[e], x[e], ssq);
+      else if (i < qn + kn) ssk = fmaf(x[e], x[e], ssk);
+    }
+  }
   for (int i = threadIdx.x; i < half; i += NT) {
     float sn, cs;
     sincosf((float)pos * p.inv_freq[i], &sn, &cs);
     cosines[i] = cs * p.magnitude;
     sines[i] = sn * p.magnitude;
   }
-  if (spread)
-    for (int i = threadIdx.x; i < p.H * p.H; i += NT) mix[i] = p.mix[i];
-  const float* row = p.src + (size_t)t * p.src_stride;
-  float ssq = 0.f, ssk = 0.f;
-  for (int i = threadIdx.x; i < qn + kn + vn; i += NT) {
-    float x = 0.f;
-    for (int s = 0; s < p.splits; ++s) x += row[(size_t)s * p.split_stride + i];
-    if (p.bias) x += p.bias[i];
-    smem[i] = x;
-    if (i < qn) ssq = fmaf(x, x, ssq);
-    else if (i < qn + kn) ssk = fmaf(x, x, ssk);
-  }
   const float inv_q = p.wq ? 1.f / sqrtf(block_sum<NT>(ssq, scratch) / (float)qn + p.eps) : 1.f;
   const float inv_k = p.wk ? 1.f / sqrtf(block_sum<NT>(ssk, scratch) / (float)kn + p.eps) : 1.f;
   __syncthreads();
-  // norm and rotation, in place: the lower entry of a rotated pair does both
-  const int per_head = half + (p.D - p.dims);
+  // norm and rotation, in place: the lower entries of rotated pairs do both
+  const int turned = half / W, per_head = turned + (p.D - p.dims) / W;
   for (int item = threadIdx.x; item < (p.H + p.G) * per_head; item += NT) {
     const int head = item / per_head, i = item - head * per_head;
-    const int e = i < half ? i : i + half;
-    float* x = smem + (size_t)head * p.D + e;
+    const int e0 = i < turned ? i * W : i * W + half;
+    float* x = q + (size_t)head * p.D + e0;
     const bool is_q = head < p.H;
     const float* w = is_q ? p.wq : p.wk;
-    if (w) w += (size_t)(is_q ? head : head - p.H) * p.D + e;
+    if (w) w += (size_t)(is_q ? head : head - p.H) * p.D + e0;
     const float inv = is_q ? inv_q : inv_k;
-    const float a = x[0] * inv * (w ? w[0] : 1.f);
-    if (i < half) {
-      const float b = x[half] * inv * (w ? w[half] : 1.f);
-      x[0] = a * cosines[i] - b * sines[i];
-      x[half] = b * cosines[i] + a * sines[i];
+    float a[W], f[W];
+    load_w<W>(x, a);
+    if (w) {
+      load_w<W>(w, f);
+#pragma unroll
+      for (int e = 0; e < W; ++e) a[e] = a[e] * inv * f[e];
+    }
+    if (i < turned) {
+      float b[W], c[W], s[W], lo[W], hi[W];
+      load_w<W>(x + half, b);
+      if (w) {
+        load_w<W>(w + half, f);
+#pragma unroll
+        for (int e = 0; e < W; ++e) b[e] = b[e] * inv * f[e];
+      }
+      load_w<W>(cosines + i * W, c);
+      load_w<W>(sines + i * W, s);
+#pragma unroll
+      for (int e = 0; e < W; ++e) {
+        lo[e] = a[e] * c[e] - b[e] * s[e];
+        hi[e] = b[e] * c[e] + a[e] * s[e];
+      }
+      store_w<W>(x, lo);
+      store_w<W>(x + half, hi);
     } else {
-      x[0] = a;
+      store_w<W>(x, a);
     }
   }
-  if (p.value_mode == 1) {
-    for (int i = threadIdx.x; i < vn; i += NT) p.v_first[(size_t)t * vn + i] = v[i];
-  } else if (p.value_mode == 2) {
-    const float l = *p.lambda;
-    for (int i = threadIdx.x; i < vn; i += NT) v[i] = (1.f - l) * v[i] + l * p.v_first[(size_t)t * vn + i];
+  if (p.value_mode) {
+    const float l = p.value_mode == 2 ? *p.lambda : 0.f;
+    float* first = p.v_first + (size_t)t * vn;
+    for (int i = threadIdx.x * W; i < vn; i += NT * W) {
+      float mine[W], theirs[W];
+      load_w<W>(v + i, mine);
+      if (p.value_mode == 1) {
+        store_w<W>(first + i, mine);
+      } else {
+        load_w<W>(first + i, theirs);
+#pragma unroll
+        for (int e = 0; e < W; ++e) mine[e] = (1.f - l) * mine[e] + l * theirs[e];
+        store_w<W>(v + i, mine);
+      }
+    }
   }
   __syncthreads();
-  const int pairs = p.P >> 1;
+  const int pieces = p.P / W;
+  // a row of n entries at ``src``, padded with zeros to P
+  auto piece = [&](const float* src, int i, int n, float (&x)[W]) {
+    if (i < n) {
+      load_w<W>(src + i, x);
+    } else {
+#pragma unroll
+      for (int e = 0; e < W; ++e) x[e] = 0.f;
+    }
+  };
   if (p.write_kv) {
     int page = -1;
     if (TL_DEBUG_OK(pos / p.page_size < p.table_width, TL_DEBUG_POSITION, pos))
@@ -165,44 +254,61 @@ qkv_prepare_kernel(const Params p, T* __restrict__ pages, T* __restrict__ q_out)
     if (TL_DEBUG_OK(page >= 0 && page < p.num_pages, TL_DEBUG_PAGE, page) && page >= 0) {
       // pages: [num_pages, 2, G, page_size, P]
       T* dst = pages + (size_t)page * 2 * p.G * p.page_size * p.P + (size_t)(pos % p.page_size) * p.P;
-      for (int item = threadIdx.x; item < 2 * p.G * pairs; item += NT) {
-        const int head = item / pairs, i = (item - head * pairs) * 2;  // key heads, then value heads
+      for (int item = threadIdx.x; item < 2 * p.G * pieces; item += NT) {
+        const int head = item / pieces, i = (item - head * pieces) * W;  // key heads, then value heads
         const bool is_v = head >= p.G;
-        const int n = is_v ? p.V : p.D;
-        const float* src = is_v ? v + (size_t)(head - p.G) * p.V : k + (size_t)head * p.D;
-        store2<T>(dst + (size_t)head * p.page_size * p.P + i, i < n ? src[i] : 0.f, i + 1 < n ? src[i + 1] : 0.f);
+        float x[W];
+        piece(is_v ? v + (size_t)(head - p.G) * p.V : k + (size_t)head * p.D, i, is_v ? p.V : p.D, x);
+        store_w<W>(dst + (size_t)head * p.page_size * p.P + i, x);
       }
     }
   }
   T* out = q_out + (size_t)t * p.q_stride;
   if (!spread) {
-    for (int item = threadIdx.x; item < p.H * pairs; item += NT) {
-      const int head = item / pairs, i = (item - head * pairs) * 2;
-      const float* src = q + (size_t)head * p.D;
-      store2<T>(out + (size_t)head * p.P + i, i < p.D ? src[i] : 0.f, i + 1 < p.D ? src[i + 1] : 0.f);
+    for (int item = threadIdx.x; item < p.H * pieces; item += NT) {
+      const int head = item / pieces, i = (item - head * pieces) * W;
+      float x[W];
+      piece(q + (size_t)head * p.D, i, p.D, x);
+      store_w<W>(out + (size_t)head * p.P + i, x);
     }
     return;
   }
   switch (p.H / p.G) {
-    case 1: spread_queries<T, 1>(p, q, mix, out); break;
-    case 2: spread_queries<T, 2>(p, q, mix, out); break;
-    case 4: spread_queries<T, 4>(p, q, mix, out); break;
-    case 8: spread_queries<T, 8>(p, q, mix, out); break;
-    default: spread_queries<T, 0>(p, q, mix, out); break;
+    case 1: spread_queries<T, NT, 1, W>(p, q, mix, out); break;
+    case 2: spread_queries<T, NT, 2, W>(p, q, mix, out); break;
+    case 4: spread_queries<T, NT, 4, W>(p, q, mix, out); break;
+    case 8: spread_queries<T, NT, 8, W>(p, q, mix, out); break;
+    default: spread_queries<T, NT, 0, W>(p, q, mix, out); break;
   }
 }
 
-template <typename T>
-int launch(const Params& p, void* pages, void* q_out, int tokens, cudaStream_t stream) {
-  const size_t floats = (size_t)p.H * p.D + (size_t)p.G * (p.D + p.V) + p.dims + (p.mix ? (size_t)p.H * p.H : 0);
-  const size_t smem = floats * sizeof(float);
-  if (smem > 200 * 1024) return TL_ERR_UNSUPPORTED;
+template <typename T, int NT, int W>
+int launch(const Params& p, void* pages, void* q_out, int tokens, size_t smem, cudaStream_t stream) {
   if (smem > 48 * 1024) {
-    const cudaError_t err = cudaFuncSetAttribute(qkv_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t err = cudaFuncSetAttribute(qkv_prepare_kernel<T, NT, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) return (int)err;
   }
-  tl::launch_kernel(qkv_prepare_kernel<T>, (unsigned)tokens, NT, smem, stream, p, (T*)pages, (T*)q_out);
+  tl::launch_kernel(qkv_prepare_kernel<T, NT, W>, (unsigned)tokens, NT, smem, stream, p, (T*)pages, (T*)q_out);
   return TL_LAUNCH_CHECK();
+}
+
+template <typename T>
+int pick(Params p, void* pages, void* q_out, int tokens, cudaStream_t stream) {
+  p.mix_floats = p.mix ? (p.H * p.H + 3) / 4 * 4 : 0;
+  const size_t half = p.dims / 2, vn = (size_t)p.G * p.V;
+  const size_t floats = p.mix_floats + (size_t)(p.H + p.G) * p.D + (vn + 3) / 4 * 4 + 2 * ((half + 3) / 4 * 4);
+  const size_t smem = floats * sizeof(float);
+  if (smem > 200 * 1024) return TL_ERR_UNSUPPORTED;
+  uintptr_t all = 0;
+  for (const void* x : {(const void*)p.src, (const void*)p.bias, (const void*)p.wq, (const void*)p.wk, (const void*)p.v_first,
+                        (const void*)pages, (const void*)q_out})
+    all |= reinterpret_cast<uintptr_t>(x);
+  // 16-byte pieces; the choice of kernel depends on sizes and alignment (and on split sums) alone, never on the batch
+  const bool wide = p.D % 4 == 0 && p.V % 4 == 0 && p.dims % 8 == 0 && p.P % 4 == 0 && p.src_stride % 4 == 0 &&
+                    p.split_stride % 4 == 0 && p.q_stride % 4 == 0 && (all & 15) == 0;
+  if (p.splits > 1)
+    return wide ? launch<T, 1024, 4>(p, pages, q_out, tokens, smem, stream) : launch<T, 1024, 1>(p, pages, q_out, tokens, smem, stream);
+  return wide ? launch<T, 256, 4>(p, pages, q_out, tokens, smem, stream) : launch<T, 256, 1>(p, pages, q_out, tokens, smem, stream);
 }
 
 }  // namespace
@@ -233,6 +339,6 @@ extern "C" int tl_qkv_prepare(const float* src, int splits, long long split_stri
   p.H = H; p.G = G; p.D = D; p.V = V; p.P = P; p.dims = dims;
   p.mix = mix; p.spread = spread; p.v_first = v_first; p.lambda = lambda; p.value_mode = value_mode;
   p.write_kv = write_kv; p.q_stride = q_stride;
-  return dtype == TL_DTYPE_F32 ? launch<float>(p, pages, q_out, tokens, stream)
-                               : launch<__nv_bfloat16>(p, pages, q_out, tokens, stream);
+  return dtype == TL_DTYPE_F32 ? pick<float>(p, pages, q_out, tokens, stream)
+                               : pick<__nv_bfloat16>(p, pages, q_out, tokens, stream);
 }

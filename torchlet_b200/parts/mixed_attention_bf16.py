@@ -43,9 +43,9 @@ def query_form(mixer, ctx, cache) -> int:
 
 def decode_splits(requests: int, keys: int, device) -> int:
     """CTAs that share the key tiles of one request: as many as fill one wave (the kernel's stages leave room for one CTA an
-    SM), no share below 64 keys.  ``keys``: the most keys a request of the step, or of the captured graph, may see."""
+    SM), no share below 96 keys.  ``keys``: the most keys a request of the step, or of the captured graph, may see."""
     index = torch.cuda.current_device() if device.index is None else device.index
-    return max(1, min(attention_bf16._sm_count(index) // max(1, requests), -(-keys // 64)))
+    return max(1, min(attention_bf16._sm_count(index) // max(1, requests), -(-keys // 96)))
 
 
 def forward(mixer, ctx, q, cache, out) -> bool:
