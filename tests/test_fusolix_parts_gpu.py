@@ -66,6 +66,10 @@ def test_streams_are_read_through_a_layer_norm_and_written_all_at_once(n, width)
     total = torch.empty(T, width, device=DEV)
     ops.hyper_collapse(got, total)
     close(total, got.sum(dim=1).cpu(), 1e-6, "the streams' sum")
+    joined = torch.empty(T, width, device=DEV)  # the write and the sum as one kernel
+    side = y.to(DEV)
+    ops.hyper_collapse(z.to(DEV), joined, write=(side, mix.to(DEV), b.to(DEV)))
+    assert torch.equal(joined, total) and not side.any()
 
 
 # ------------------------------------------------------------- input convolution

@@ -45,7 +45,7 @@ def plan_groups(needs: list, num_pages: int) -> tuple[list[GroupSpec], dict]:
         members[key].append(need.entry)
     groups, where = [], {}
     for g, key in enumerate(keys):
-        groups.append(GroupSpec(key[0], key[1], key[2], tuple(members[key]), num_pages, planes=key[3], keep_first=key[4]))
+        groups.append(GroupSpec(key[0], key[1], key[2], tuple(members[key]), num_pages, planes=key[3], keep_first=key[4] if len(key) > 4 else 0))
         for i, entry in enumerate(members[key]):
             where[entry] = (g, i)
     return groups, where

@@ -6,7 +6,8 @@
 //
 // Kernels (all float32 inside; T is the type of what a sub-layer reads):
 //   fanout        z[t, s] = acc[t] for every s                       (the streams start equal)
-//   collapse      acc[t] = sum_s z[t, s], ascending s
+//   collapse      acc[t] = sum_s z[t, s], ascending s; it can take the last sub-layer's write along (the new streams are
+//                 summed from registers and never stored: nobody reads them behind the sum)
 //   read_norm     one block a token: u, then (u - mean) / sqrt(var + eps) * w + b (``centre``) or
 //                 u / sqrt(mean(u^2) + eps) * w (no centring); h float32, or T when no convolution follows.
 //                 It can take the WRITE of the sub-layer before into the same pass, and, in a step of single tokens,
@@ -82,6 +83,51 @@ template <int V> __device__ __forceinline__ void store_v(__nv_bfloat16* p, const
   } else {
     *p = __float2bfloat16_rn(v[0]);
   }
+}
+
+// The sum of the streams as the write of the last sub-layer would leave them; every sum as in write_kernel and
+// collapse_kernel.  V consecutive channels a thread.
+template <int V>
+__global__ void __launch_bounds__(256)
+write_collapse_kernel(const float* __restrict__ z, float* __restrict__ y, const float* __restrict__ mix,
+                      const float* __restrict__ b, float* __restrict__ acc, int n, int width, size_t total) {
+  tl::pdl_launch_dependents();
+  tl::pdl_wait();
+  __shared__ float s_mix[MAX_STREAMS * MAX_STREAMS], s_b[MAX_STREAMS];
+  if (threadIdx.x < n * n) s_mix[threadIdx.x] = mix[threadIdx.x];
+  if (threadIdx.x < n) s_b[threadIdx.x] = b[threadIdx.x];
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  const bool live = i < total;
+  const size_t t = live ? i / width : 0, c = live ? i - t * width : 0;
+  float old[MAX_STREAMS][V], add[V], sum[V];
+  if (live) {
+#pragma unroll
+    for (int s = 0; s < MAX_STREAMS; ++s)
+      if (s < n)
+        load_v<V>(z + (t * n + s) * width + c, old[s]);
+    load_v<V>(y + i, add);
+  }
+  __syncthreads();
+  if (!live) return;
+#pragma unroll
+  for (int e = 0; e < V; ++e) sum[e] = 0.f;
+#pragma unroll
+  for (int to = 0; to < MAX_STREAMS; ++to) {
+    if (to < n) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        float v = 0.f;
+#pragma unroll
+        for (int s = 0; s < MAX_STREAMS; ++s)
+          if (s < n) v = fmaf(s_mix[s * n + to], old[s][e], v);
+        sum[e] += fmaf(s_b[to], add[e], v);
+      }
+    }
+  }
+  store_v<V>(acc + i, sum);
+#pragma unroll
+  for (int e = 0; e < V; ++e) add[e] = 0.f;
+  store_v<V>(y + i, add);  // behind the stores that needed its old value (see read_norm_kernel)
 }
 
 // NT threads a block: 256, or 512 for wide rows, where a thread then walks few channels (a step of few tokens is a
@@ -334,10 +380,22 @@ int tl_hyper_fanout(const float* acc, float* z, int tokens, int n, int width, cu
   return TL_LAUNCH_CHECK();
 }
 
-int tl_hyper_collapse(const float* z, float* acc, int tokens, int n, int width, cudaStream_t stream) {
+// y, mix, b (or nullptr): the write of the last sub-layer, z_t <- sum_s mix[s, t] z_s + b_t y, comes first; z stays, y is
+// left zeroed.
+int tl_hyper_collapse(const float* z, float* acc, int tokens, int n, int width, float* y, const float* mix, const float* b,
+                      cudaStream_t stream) {
   const size_t total = (size_t)tokens * width;
   if (total == 0) return 0;
   if (n <= 0) return TL_ERR_UNSUPPORTED;
+  if (y) {
+    if (n > MAX_STREAMS || !mix || !b) return TL_ERR_UNSUPPORTED;
+    const uintptr_t all = (uintptr_t)z | (uintptr_t)y | (uintptr_t)acc;
+    if (width % 4 == 0 && (all & 15) == 0)
+      tl::launch_kernel(write_collapse_kernel<4>, (unsigned)((total / 4 + 255) / 256), 256, 0, stream, z, y, mix, b, acc, n, width, total);
+    else
+      tl::launch_kernel(write_collapse_kernel<1>, (unsigned)((total + 255) / 256), 256, 0, stream, z, y, mix, b, acc, n, width, total);
+    return TL_LAUNCH_CHECK();
+  }
   tl::launch_kernel(collapse_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, z, acc, n, width, total);
   return TL_LAUNCH_CHECK();
 }

@@ -19,7 +19,32 @@ using namespace tl;
 
 constexpr int NT = 256;
 
-template <typename T>
+// V consecutive channels: 4 where width and addresses allow 16-byte pieces (8-byte ones of the bfloat16 tables), else 1.
+template <int V> __device__ __forceinline__ void load_v(const float* p, float (&out)[V]) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    out[0] = v.x; out[1] = v.y; out[2] = v.z; out[3] = v.w;
+  } else {
+    out[0] = *p;
+  }
+}
+template <int V> __device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&out)[V]) {
+  if constexpr (V == 4) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    out[0] = __uint_as_float(raw.x << 16);
+    out[1] = __uint_as_float(raw.x & 0xffff0000u);
+    out[2] = __uint_as_float(raw.y << 16);
+    out[3] = __uint_as_float(raw.y & 0xffff0000u);
+  } else {
+    out[0] = __bfloat162float(*p);
+  }
+}
+template <int V> __device__ __forceinline__ void store_v(float* p, const float (&v)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else *p = v[0];
+}
+
+template <typename T, int V>
 __global__ void __launch_bounds__(NT)
 token_embed_kernel(const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ ids,
                    const int* __restrict__ positions, const int* __restrict__ token_req, const int* __restrict__ req_indptr,
@@ -55,30 +80,50 @@ token_embed_kernel(const T* __restrict__ table, const T* __restrict__ pairs, con
   const T* row = table + (size_t)(ok ? id : 0) * width;
   const T* pair = pairs ? pairs + (size_t)pair_row * width : nullptr;
   float sum = 0.f;
-  for (int c = threadIdx.x; c < width; c += NT) {
-    float v = ok ? to_float(row[c]) * scale : 0.f;
-    if (pair) v += to_float(pair[c]);
-    x[c] = v;
-    sum += v;
+  for (int c = threadIdx.x * V; c < width; c += NT * V) {
+    float v[V];
+    load_v<V>(row + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v[e] = ok ? v[e] * scale : 0.f;
+    if (pair) {
+      float w[V];
+      load_v<V>(pair + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] += w[e];
+    }
+    store_v<V>(x + c, v);
+#pragma unroll
+    for (int e = 0; e < V; ++e) sum += v[e];
   }
   float mean = 0.f, inv = 1.f;
   if (weight) {
     if (centre) mean = block_sum<NT>(sum, scratch) / (float)width;
     float ss = 0.f;
-    for (int c = threadIdx.x; c < width; c += NT) {  // a thread reads back what it wrote itself
-      const float d = x[c] - mean;
-      ss = fmaf(d, d, ss);
+    for (int c = threadIdx.x * V; c < width; c += NT * V) {  // a thread reads back what it wrote itself
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float d = x[c + e] - mean;
+        ss = fmaf(d, d, ss);
+      }
     }
     inv = 1.f / sqrtf(block_sum<NT>(ss, scratch) / (float)width + eps);
   }
   float* o = out + (size_t)t * streams * width;
-  for (int c = threadIdx.x; c < width; c += NT) {
-    float v = x[c];
+  for (int c = threadIdx.x * V; c < width; c += NT * V) {
+    float v[V];
+    load_v<V>(x + c, v);
     if (weight) {
-      v = (v - mean) * inv * weight[c];
-      if (bias) v += bias[c];
+      float w[V];
+      load_v<V>(weight + c, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[e] = (v[e] - mean) * inv * w[e];
+      if (bias) {
+        load_v<V>(bias + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] += w[e];
+      }
     }
-    for (int s = 0; s < streams; ++s) o[(size_t)s * width + c] = v;
+    for (int s = 0; s < streams; ++s) store_v<V>(o + (size_t)s * width + c, v);
   }
 }
 
@@ -102,7 +147,16 @@ extern "C" int tl_token_embed(const void* table, const void* pairs, int dtype, c
                       slots, last, max_slots, buckets, mul_prev, mul_cur, weight, bias, eps, centre, out, streams, width,
                       vocab, scale);
   };
-  if (dtype == TL_DTYPE_F32) run(token_embed_kernel<float>, (const float*)table, (const float*)pairs);
-  else run(token_embed_kernel<__nv_bfloat16>, (const __nv_bfloat16*)table, (const __nv_bfloat16*)pairs);
+  const uintptr_t all = (uintptr_t)table | (uintptr_t)pairs | (uintptr_t)weight | (uintptr_t)bias | (uintptr_t)out;
+  const bool wide = width % 4 == 0 && (all & 15) == 0;
+  const float *table32 = (const float*)table, *pairs32 = (const float*)pairs;
+  const __nv_bfloat16 *table16 = (const __nv_bfloat16*)table, *pairs16 = (const __nv_bfloat16*)pairs;
+  if (dtype == TL_DTYPE_F32) {
+    if (wide) run(token_embed_kernel<float, 4>, table32, pairs32);
+    else run(token_embed_kernel<float, 1>, table32, pairs32);
+  } else {
+    if (wide) run(token_embed_kernel<__nv_bfloat16, 4>, table16, pairs16);
+    else run(token_embed_kernel<__nv_bfloat16, 1>, table16, pairs16);
+  }
   return TL_LAUNCH_CHECK();
 }

@@ -226,7 +226,7 @@ _SIGNATURES = {
     },
     "hyper": {
         "tl_hyper_fanout": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-        "tl_hyper_collapse": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "tl_hyper_collapse": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
         "tl_hyper_read_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                c_int, c_void_p],
@@ -721,12 +721,17 @@ def hyper_fanout(acc, z) -> None:
     _check(_fn("hyper", "tl_hyper_fanout")(acc.data_ptr(), z.data_ptr(), tokens, n, width, _stream()), "hyper_fanout")
 
 
-def hyper_collapse(z, acc) -> None:
-    """acc[t] = sum_s z[t, s] (ascending s)."""
-    _need_cuda(acc, z)
+def hyper_collapse(z, acc, write=None) -> None:
+    """acc[t] = sum_s z[t, s] (ascending s).  ``write`` = (y, mix, b): of the streams as ``hyper_write`` of these would leave
+    them (z stays as it is, y is left zeroed)."""
+    y, mix, b = write if write is not None else (None, None, None)
+    _need_cuda(acc, z, y, mix, b)
+    assert y is None or (y.dtype == mix.dtype == b.dtype == torch.float32 and y.is_contiguous() and y.shape == acc.shape
+                         and mix.is_contiguous() and mix.shape == (z.shape[1], z.shape[1]) and b.numel() == z.shape[1])
     tokens, n, width = z.shape
     assert acc.dtype == z.dtype == torch.float32 and acc.is_contiguous() and z.is_contiguous() and acc.shape == (tokens, width)
-    _check(_fn("hyper", "tl_hyper_collapse")(z.data_ptr(), acc.data_ptr(), tokens, n, width, _stream()), "hyper_collapse")
+    _check(_fn("hyper", "tl_hyper_collapse")(z.data_ptr(), acc.data_ptr(), tokens, n, width, _ptr(y), _ptr(mix), _ptr(b),
+                                             _stream()), "hyper_collapse")
 
 
 def hyper_read_norm(z, a, weight, bias, eps: float, out, centre: bool = True, rows=None, write=None, conv=None) -> None:

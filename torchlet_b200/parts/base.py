@@ -48,7 +48,8 @@ class KVSpec:
     keep_first: int = 0
 
     def group_key(self) -> tuple:
-        return (self.num_kv_heads, self.head_dim, self.window, self.planes, self.keep_first if self.window is not None else 0)
+        key = (self.num_kv_heads, self.head_dim, self.window, self.planes)
+        return key + (self.keep_first,) if self.keep_first and self.window is not None else key
 
 
 @dataclass(frozen=True)

@@ -164,8 +164,9 @@ class LayeredModel:
         # several residual streams a token, all equal to the embedding at the start; their sum at the end
         for i, entry in enumerate(self.spec.schedule):
             self.blocks[entry.layer].forward(ctx, z, caches[i])
+        write = ctx.take_write(z)  # the last sub-layer's, joined with the sum
         ctx.flush_pending()
-        ops.hyper_collapse(z, acc)
+        ops.hyper_collapse(z, acc, write)
         return acc
 
     def _embeds_at_once(self) -> bool:
