@@ -245,3 +245,44 @@ def test_trace_replay_chooses_the_model_by_its_configuration(tmp_path):
     V = cases.CASES[name]["vocab"]
     got = torch.cat([torch.from_numpy(np.fromfile(out / f"{i}.f32", dtype="<f4").reshape(-1, V)) for i in range(3)])
     cases.assert_close(got, want[[0, 19, 20, 29]], "float32", "trace replay")
+
+
+@pytest.mark.parametrize("graph", [False, True])
+@pytest.mark.parametrize("name,dtype", [("P", "float32"), ("P", "bfloat16"), ("R", "bfloat16")])
+def test_scratch_memory_full_of_nan(name, dtype, graph):
+    """Every scratch buffer starts as NaN: whatever a kernel reads without having written it shows."""
+    from test_poisoned_memory_gpu import poison
+
+    name = cases.variant(name, dtype)
+    poison(1000)
+    runner = cases.make_runner(name, dtype, cuda_graph=graph)
+    ids, want = cases.plain_logits(name, 150, 31)
+    for cuts in ([150], [118] + [1] * 32, [2, 7, 1, 40, 3, 2, 60, 1, 34]):
+        poison(200)
+        cases.assert_close(cases.replay(runner, "r", ids, cuts), want, dtype, f"{name} in {len(cuts)} portions")
+
+
+def test_first_values_come_from_the_first_mixing_layer_of_the_same_step():
+    """Two requests in one step, portions and single tokens: each token is mixed with its own first values (a model whose
+    value mixing is turned off gives other logits)."""
+    from torchlet_b200.engine import StepEntry
+
+    seqs = [cases.plain_logits("P", n, 80 + n) for n in (40, 25)]
+    runner = cases.make_runner("P", "float32")
+    for r in (0, 1):
+        runner.admit(r)
+    at, got = [0, 0], [[], []]
+    for sizes in ((9, 1), (1, 12), (1, 1), (20, 3), (9, 8)):
+        entries = [StepEntry(r, seqs[r][0][at[r]:at[r] + n], list(range(n))) for r, n in enumerate(sizes)]
+        logits, row = runner.step(entries).cpu(), 0
+        for r, n in enumerate(sizes):
+            got[r].append(logits[row:row + n].clone())
+            row, at[r] = row + n, at[r] + n
+    for r in (0, 1):
+        cases.assert_close(torch.cat(got[r]), seqs[r][1], "float32", f"request {r}")
+    off = dict(cases.weights_for("P"))
+    for key in off:
+        if key.endswith(".vmix"):
+            off[key] = torch.zeros(())
+    other = plain_lidizen.forward(off, cases.CASES["P"], seqs[0][0]).float()
+    assert (other - seqs[0][1]).abs().max() > 0.05 * seqs[0][1].abs().max()
