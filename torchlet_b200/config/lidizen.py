@@ -182,13 +182,16 @@ class LidizenConfig:
                 value_mix = "later" if mixed_before else "first"
                 mixed_before = True
             feed_forward = self._feed_forward(layer.get("mlp"))
-            norms = [NormSlot("mixer_norm", norm, "norm1")]
+            norms, unused = [NormSlot("mixer_norm", norm, "norm1")], ()
             if feed_forward is not None:
                 norms.append(NormSlot("feed_forward_norm", norm, "norm2"))
+            else:  # a checkpoint may carry the second sub-layer's norm and connections all the same
+                n = self.streams
+                unused = (("norm2", (W,)), ("hc2.in", (n,)), ("hc2.out", (n,)), ("hc2.mix", (n, n)))
             layers.append(LayerSpec(
                 prefix=f"l{i}.", block="hyper_connected", mixer=self._mixer(layer["mixer"], value_mix),
                 feed_forward=feed_forward, norms=tuple(norms), mixer_prefix="mix.", feed_forward_prefix="mlp.",
-                block_params={"streams": self.streams, "taps": None, "connections": ("hc1.", "hc2.")}))
+                block_params={"streams": self.streams, "taps": None, "connections": ("hc1.", "hc2."), "unused": unused}))
             schedule.append(ScheduleEntry(layer=i))
         pairs = TokenPairs("bigram", *self.bigram) if self.bigram is not None else None
         spec = ModelSpec(

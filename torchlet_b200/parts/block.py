@@ -154,7 +154,8 @@ class HyperConnectedBlock(Block):
 
     Parameters: ``streams`` (n), ``taps`` (None: no convolution), ``connections`` (the tensor prefixes of the two
     sub-layers' a, b, M below the layer's: ``<c>in`` [n], ``<c>out`` [n], ``<c>mix`` [n, n]), ``convolutions`` (the
-    names of the two convolution weights, [width, taps])."""
+    names of the two convolution weights, [width, taps]), ``unused`` ((name, shape) of tensors that may stand in the
+    checkpoint without being read)."""
 
     norm_roles = ("mixer_norm",)
     SUBLAYERS = ("mixer", "feed_forward")
@@ -198,6 +199,8 @@ class HyperConnectedBlock(Block):
                     TensorSpec(p + "mix", (n, n), init="eye")]
             if convolution is not None:
                 out.append(TensorSpec(layer.prefix + convolution, (width, int(taps))))
+        # tensors a checkpoint may carry for a sub-layer the layer does not have; nothing reads them
+        out += [TensorSpec(layer.prefix + name, tuple(shape), optional=True) for name, shape in layer.block_params.get("unused", ())]
         return out
 
     def load(self, tensors: dict, layer, device, dtype) -> None:
